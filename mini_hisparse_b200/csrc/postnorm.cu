@@ -221,7 +221,8 @@ __global__ void qknorm_rope_append_kernel(const float* __restrict__ qkv, int nsp
                                           int table_width, const float* __restrict__ inv_freq, int rdim,
                                           QT* __restrict__ q_out, CT* __restrict__ cache, int nq, int nkv, int dk,
                                           int dv, int P, int num_pages, int has_kv, int* __restrict__ status,
-                                          int per_head, float v_eps, size_t page_extra) {
+                                          int per_head, float v_eps, size_t page_extra, float temp_coef,
+                                          double temp_every, float v_scale) {
     extern __shared__ float sh[];            // q row, k row, cos, sin (and the v row, if it is normalised)
     __shared__ float scratch[33];
     pdl_launch_dependents();
@@ -260,7 +261,10 @@ __global__ void qknorm_rope_append_kernel(const float* __restrict__ qkv, int nsp
             float ss = 0.f;
             for (int e = lane; e < dk; e += 32) ss += row[e] * row[e];
             const float r = 1.f / sqrtf(warp_sum(ss) / (float)dk + eps);
-            for (int e = lane; e < dk; e += 32) row[e] = row[e] * r * w[e];
+            // a temperature that grows with the position, on q alone: 1 + coef ln(floor((pos + 1) / every) + 1)
+            const float f = head < nq && temp_coef != 0.f
+                                ? 1.f + temp_coef * log1pf((float)floor((double)(pos + 1) / temp_every)) : 1.f;
+            for (int e = lane; e < dk; e += 32) row[e] = row[e] * r * (w ? w[e] : 1.f) * f;
         }
     } else {
         const float tq = block_sum(ssq, scratch);
@@ -319,7 +323,7 @@ __global__ void qknorm_rope_append_kernel(const float* __restrict__ qkv, int nsp
         for (int i = threadIdx.x; i < vw; i += blockDim.x) {
             const int g = i / dv, e = i - g * dv;
             page_v[((size_t)g * P + within) * dv + e] =
-                from_float<CT>(v_eps > 0.f ? vs[i] : load_parts(qkv, base + qw + kw + i, nsplit, split_stride));
+                from_float<CT>(v_scale * (v_eps > 0.f ? vs[i] : load_parts(qkv, base + qw + kw + i, nsplit, split_stride)));
         }
     }
 }
@@ -417,14 +421,20 @@ MHB_EXPORT int mhb_gated_rmsnorm(const float* o, const float* gate, int gate_nsp
 
 // per_head: the two norms run over each head alone, with weights [dk] that the heads share, instead of over the whole
 // projections.  v_eps > 0: every head's value is divided by its root mean square (with that eps) before it is stored.
-// page_extra: elements of a page behind its keys and values (left alone here).
+// page_extra: elements of a page behind its keys and values (left alone here).  temp_coef != 0 (with per_head): q is
+// multiplied by 1 + temp_coef ln(floor((position + 1) / temp_every) + 1).  v_scale: a factor on the stored values.
+// With per_head the weights may be null (norms without a weight).
 MHB_EXPORT int mhb_qknorm_rope_append_opts(const float* qkv, int nsplit, long long split_stride, int ld,
                                       const float* q_weight, const float* k_weight, float eps, const int* positions,
                                       const int* tok_seg, const int* block_table, int table_width,
                                       const float* inv_freq, int rdim, void* q_out, void* cache, int dtype, int T,
                                       int nq, int nkv, int dk, int dv, int P, int num_pages, int has_kv, int* status,
-                                      int per_head, float v_eps, long long page_extra, cudaStream_t stream) {
+                                      int per_head, float v_eps, long long page_extra, float temp_coef,
+                                      double temp_every, float v_scale, cudaStream_t stream) {
     if (T <= 0) return 0;
+    if (!per_head && (!q_weight || (has_kv && !k_weight) || temp_coef != 0.f))
+        return fail("qknorm_rope_append: norms over whole projections have weights and no temperature");
+    if (temp_coef != 0.f && !(temp_every > 0.)) return fail("qknorm_rope_append: a temperature needs a positive step");
     if (rdim < 0 || rdim > dk || (rdim & 1)) return fail("qknorm_rope_append: %d rotated elements of a head of %d", rdim, dk);
     const int qw = nq * dk, kw = has_kv ? nkv * dk : 0;
     const size_t smem = sizeof(float) * ((size_t)qw + kw + rdim + (v_eps > 0.f && has_kv ? (size_t)nkv * dv : 0));
@@ -434,7 +444,7 @@ MHB_EXPORT int mhb_qknorm_rope_append_opts(const float* qkv, int nsplit, long lo
         launch_kernel(kern, dim3(T), dim3(row_threads(qw + kw)), smem, stream, qkv, nsplit, (size_t)split_stride, ld,
                       q_weight, k_weight, eps, positions, tok_seg, block_table, table_width, inv_freq, rdim,
                       (CT*)q_out, (CT*)cache, nq, nkv, dk, dv, P, num_pages, has_kv, status, per_head, v_eps,
-                      (size_t)page_extra);
+                      (size_t)page_extra, temp_coef, temp_every, v_scale);
     });
     return check_launch("qknorm_rope_append");
 }
@@ -447,5 +457,5 @@ MHB_EXPORT int mhb_qknorm_rope_append(const float* qkv, int nsplit, long long sp
                                       cudaStream_t stream) {
     return mhb_qknorm_rope_append_opts(qkv, nsplit, split_stride, ld, q_weight, k_weight, eps, positions, tok_seg,
                                        block_table, table_width, inv_freq, rdim, q_out, cache, dtype, T, nq, nkv, dk, dv,
-                                       P, num_pages, has_kv, status, 0, 0.f, 0, stream);
+                                       P, num_pages, has_kv, status, 0, 0.f, 0, 0.f, 1., 1.f, stream);
 }

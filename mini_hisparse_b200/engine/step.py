@@ -62,6 +62,7 @@ class _Layout:
         self.positions = take(T)
         self.tok_seg = take(T)
         self.seg_slot = take(S)
+        self.seg_offset = take(S + 1)
         self.rows = take(R)
         self.tables = [take(S * w) for w in widths]
         self.plans = [{name: take(n) for name, n in caps.items()} for caps in plan_caps]
@@ -207,7 +208,9 @@ class BatchBuilder:
             positions[sl] = np.arange(s.start, s.start + s.count, dtype=np.int32)
             tok_seg[sl] = si
             buf[layout.seg_slot + si] = s.slot
+            buf[layout.seg_offset + si] = s.offset
             rows.extend(s.offset + w for w in e.want)
+        buf[layout.seg_offset + len(segments)] = T
         if len(rows) > layout.R:
             raise StepError("more rows wanted than the layout holds")
         buf[layout.rows : layout.rows + len(rows)] = rows
@@ -233,6 +236,8 @@ class BatchBuilder:
         buf[layout.positions : layout.positions + B] = starts
         buf[layout.tok_seg : layout.tok_seg + B] = ar
         buf[layout.seg_slot : layout.seg_slot + B] = slots
+        buf[layout.seg_offset : layout.seg_offset + B] = ar
+        buf[layout.seg_offset + B] = B
         buf[layout.rows : layout.rows + B] = ar
         for gi, g in enumerate(self.cache.page_groups):
             width = layout.widths[gi]
@@ -258,6 +263,7 @@ class BatchBuilder:
             "positions": v(layout.positions, T),
             "tok_seg": v(layout.tok_seg, T),
             "seg_slot": v(layout.seg_slot, S),
+            "seg_offset": v(layout.seg_offset, S + 1),
             "rows": v(layout.rows, R) if R else None,
             "tables": [v(layout.tables[gi], S * w).view(S, w) for gi, w in enumerate(layout.widths)],
             "plans": plans,
@@ -284,7 +290,7 @@ class BatchBuilder:
         return StepContext(
             rt=rt, ws=ws, T=sum(s.count for s in segments), segments=segments,
             tokens=views["tokens"], positions=views["positions"], tok_seg=views["tok_seg"],
-            seg_slot=views["seg_slot"], status=status,
+            seg_slot=views["seg_slot"], status=status, seg_offset=views["seg_offset"],
         )
 
     def cache_view(self, user: int, views: dict, writable: bool = True) -> CacheView | None:
@@ -317,6 +323,9 @@ class ModelRunner:
         self.batch = BatchBuilder(cache, self.device, sm_count)
         for i, entry in enumerate(model.spec.order):
             self.batch.add_user(model.entry_cache[i], model.blocks[entry.layer])
+        # memory beside that: (name, user) per run entry
+        self.sides = [[(name, self.batch.add_user(at, model.blocks[entry.layer].side_user(name)))
+                       for name, at in model.entry_sides[i].items()] for i, entry in enumerate(model.spec.order)]
         self.sm_count = self.batch.sm_count
         self.ws = Workspace(self.device)
         self.status = torch.zeros(1, dtype=torch.int32, device=self.device)
@@ -342,8 +351,15 @@ class ModelRunner:
         build.build_all(model.kernel_modules())
 
     def _cache_views(self, views) -> list[CacheView | None]:
-        return [self.batch.cache_view(i, views, writable=entry.cache_of is None)
-                for i, entry in enumerate(self.model.spec.order)]
+        out = []
+        for i, entry in enumerate(self.model.spec.order):
+            view = self.batch.cache_view(i, views, writable=entry.cache_of is None)
+            if self.sides[i]:
+                if view is None:
+                    view = CacheView(None, -1, -1, True, None)
+                view.sides = {name: self.batch.cache_view(user, views) for name, user in self.sides[i]}
+            out.append(view)
+        return out
 
     # ---- the step -----------------------------------------------------------------------------
     @torch.inference_mode()

@@ -7,7 +7,7 @@ device, or a size is outside what the kernel takes.
 from __future__ import annotations
 
 import ctypes
-from ctypes import c_float, c_int, c_longlong, c_void_p
+from ctypes import c_double, c_float, c_int, c_longlong, c_void_p
 
 import torch
 
@@ -166,14 +166,16 @@ def gated_rmsnorm(o, weight, eps, out, gate=None, gate_nsplit=1, gate_split_stri
 
 def qknorm_rope_append(qkv, q_weight, k_weight, eps, positions, tok_seg, block_table, inv_freq, rotary_dim, q_out,
                        cache, *, nq, nkv, dk, dv, page_size, has_kv=True, nsplit=1, split_stride=0, status=None,
-                       per_head=False, v_eps=0.0, page_extra=0):
+                       per_head=False, v_eps=0.0, page_extra=0, q_temp=None, v_scale=1.0):
     """RMS norm over the whole q projection and over the whole k projection, rotation of the first
     ``rotary_dim`` elements of every head (pairs (i, i + rotary_dim/2)), q to ``q_out`` [T, nq dk], k and v
     into the pages of ``cache`` (one layer's pool; a page holds [nkv][P][dk] keys then [nkv][P][dv] values).
     ``qkv`` float32 [.., T, ld] holds [q | k | v | ...] per row; with ``has_kv`` False it holds [q | ...]
     and nothing is appended.  ``per_head``: the norms run over each head alone with weights [dk] shared by the
     heads.  ``v_eps`` > 0: every head's value is divided by its root mean square before it is stored.
-    ``page_extra``: elements of a page behind its keys and values, which this kernel leaves alone."""
+    ``page_extra``: elements of a page behind its keys and values, which this kernel leaves alone.  With ``per_head``
+    the weights may be None, and ``q_temp`` = (coef, every) multiplies q by
+    1 + coef ln(floor((position + 1) / every) + 1).  ``v_scale``: a factor on the stored values."""
     lib = build.load("postnorm")
     T = q_out.shape[0]
     if qkv.dtype != torch.float32 or qkv.stride(-1) != 1:
@@ -188,7 +190,8 @@ def qknorm_rope_append(qkv, q_weight, k_weight, eps, positions, tok_seg, block_t
         _ptr(inv_freq), c_int(rotary_dim), _ptr(q_out), _ptr(cache if has_kv else None), c_int(dtype_code(q_out.dtype)),
         c_int(T), c_int(nq), c_int(nkv), c_int(dk), c_int(dv), c_int(page_size),
         c_int(cache.shape[0] if has_kv else 0), c_int(1 if has_kv else 0), _ptr(status), c_int(1 if per_head else 0),
-        c_float(v_eps or 0.0), c_longlong(page_extra), _stream()),
+        c_float(v_eps or 0.0), c_longlong(page_extra), c_float(q_temp[0] if q_temp else 0.0),
+        c_double(q_temp[1] if q_temp else 1.0), c_float(v_scale), _stream()),
         "qknorm_rope_append")
 
 
@@ -1222,3 +1225,163 @@ def delta_scan(q, k, v, beta, decay, state, out, tok_seg, seg_slot, positions, *
                                    c_longlong(state.stride(0)), _ptr(out), _ptr(tok_seg), _ptr(seg_slot), _ptr(positions),
                                    c_int(T), c_int(S), c_int(heads), c_int(kv_heads), c_int(dk), c_int(dv),
                                    c_int(1 if writable else 0), _stream()), "delta_scan")
+
+
+# ---- convolutions over time and recurrences whose gates read the current token (csrc/timeconv.cu, selscan.cu) ----
+def _seg_args(ctx):
+    return _ptr(ctx.seg_offset), _ptr(ctx.seg_slot), _ptr(ctx.positions)
+
+
+def _keep_args(keep, rows: int, channels: int, what: str):
+    """(pointer, stride between slots) of the inputs a slot keeps: float32 [slots, rows, channels] with dense rows."""
+    if rows == 0:
+        return c_void_p(0), c_longlong(0)
+    if keep is None or keep.dtype != torch.float32 or keep.numel() < keep.shape[0] * rows * channels:
+        raise KernelError(f"{what}: a slot keeps {rows} x {channels} float32 inputs")
+    if not keep[0].is_contiguous():
+        raise KernelError(f"{what}: a slot's kept inputs must be dense")
+    return _ptr(keep), c_longlong(keep.stride(0))
+
+
+def _taps(taps, what: str):
+    """Filters as the kernels read them: contiguous float32 [taps, channels]."""
+    if taps.dtype != torch.float32 or not taps.is_contiguous():
+        raise KernelError(f"{what}: the filters are contiguous float32 [taps, channels]")
+    return taps.shape
+
+
+def stream_conv(x, alpha, weight, shift, taps, keep, ctx, out, *, delta=None, delta2=None, x_out=None, writable=True):
+    """v = x + delta + delta2 (float32, to ``x_out``, another buffer than x); h = tanh(alpha v) weight + shift;
+    out[t] = h_t + sum_j taps[j] h_(t - taps + 1 + j) per channel, with a segment's earlier inputs from ``keep`` [slots,
+    taps - 1, C], where its last ones go.  ``ctx``: the step (segments, slots, positions)."""
+    lib = build.load("timeconv")
+    T, C = x.shape
+    ntaps, _ = _taps(taps, "stream_conv")
+    if x.dtype != torch.float32 or not x.is_contiguous() or not out.is_contiguous():
+        raise KernelError("stream_conv: the stream is contiguous float32, the output contiguous")
+    if delta is None and delta2 is not None:
+        delta, delta2 = delta2, None
+    if _delta_dtype(delta, delta2) != F32:
+        raise KernelError("stream_conv: pending products are float32")
+    a, b = _delta_args(delta), _delta_args(delta2)
+    _check(lib, lib.mhb_stream_conv(_ptr(x), *a, *b, _ptr(x_out), _ptr(alpha), _ptr(weight), _ptr(shift), _ptr(taps),
+                                    *_keep_args(keep, ntaps - 1, C, "stream_conv"), *_seg_args(ctx), _ptr(out),
+                                    c_int(dtype_code(out.dtype)), c_int(T), c_int(len(ctx.segments)), c_int(ctx.longest),
+                                    c_int(C), c_int(ntaps), c_int(1 if writable else 0), _stream()), "stream_conv")
+
+
+def rows_conv(h, taps, keep, ctx, out, *, writable=True):
+    """out[t] = h_t + sum_j taps[j] h_(t - taps + 1 + j) for rows that are already normalised (see stream_conv)."""
+    lib = build.load("timeconv")
+    T, C = h.shape
+    ntaps, _ = _taps(taps, "rows_conv")
+    if h.dtype != out.dtype or not h.is_contiguous() or not out.is_contiguous():
+        raise KernelError("rows_conv: input and output are contiguous and of one dtype")
+    _check(lib, lib.mhb_rows_conv(_ptr(h), c_int(dtype_code(h.dtype)), _ptr(taps),
+                                  *_keep_args(keep, ntaps - 1, C, "rows_conv"), *_seg_args(ctx), _ptr(out), c_int(T),
+                                  c_int(len(ctx.segments)), c_int(ctx.longest), c_int(C), c_int(ntaps),
+                                  c_int(1 if writable else 0), _stream()), "rows_conv")
+
+
+def product_conv(proj, c0, taps, bias, keep, ctx, out, *, out32=None, writable=True):
+    """out = silu(conv + bias) of columns c0 .. of the float32 Product ``proj``; the kept inputs are the columns before
+    the convolution.  ``out32``: the same rows in float32."""
+    lib = build.load("timeconv")
+    T, C = out.shape
+    ntaps, _ = _taps(taps, "product_conv")
+    z = proj.tensor[..., c0:]
+    if z.dtype != torch.float32 or not out.is_contiguous() or (out32 is not None and not out32.is_contiguous()):
+        raise KernelError("product_conv: the product is float32, the outputs contiguous")
+    _check(lib, lib.mhb_product_conv(*_parts_args(z, proj.nsplit, proj.split_stride), c_int(z.stride(-2)), _ptr(taps),
+                                     _ptr(bias), *_keep_args(keep, ntaps - 1, C, "product_conv"), *_seg_args(ctx), _ptr(out),
+                                     c_int(dtype_code(out.dtype)), _ptr(out32), c_int(T), c_int(len(ctx.segments)),
+                                     c_int(ctx.longest), c_int(C), c_int(ntaps), c_int(1 if writable else 0), _stream()),
+           "product_conv")
+
+
+def dyt_rows(x, alpha, weight, shift, out, *, delta=None, delta2=None, rows=None):
+    """out[r] = tanh(alpha v) weight + shift with v = x[s] + delta[s] + delta2[s], s = rows[r] or r; without ``rows`` and
+    with a delta the sum is written back to ``x``."""
+    lib = build.load("timeconv")
+    R, H = out.shape
+    if x.dtype != torch.float32 or not x.is_contiguous() or not out.is_contiguous():
+        raise KernelError("dyt_rows: the stream is contiguous float32, the output contiguous")
+    if _delta_dtype(delta, delta2) != F32:
+        raise KernelError("dyt_rows: pending products are float32")
+    _check(lib, lib.mhb_dyt_rows(_ptr(x), *_delta_args(delta), *_delta_args(delta2), _ptr(alpha), _ptr(weight), _ptr(shift),
+                                 _ptr(rows), _ptr(out), c_int(dtype_code(out.dtype)), c_int(R), c_int(H), _stream()),
+           "dyt_rows")
+
+
+def stream_shift(x, row, *, delta=None, table=None, tokens=None, scale=1.0):
+    """x[t] += delta[t] + table[tokens[t]] * scale + row, in float32 (``table`` None: without that term)."""
+    lib = build.load("timeconv")
+    T, H = x.shape
+    if x.dtype != torch.float32 or not x.is_contiguous() or row.dtype != torch.float32 or row.numel() != H:
+        raise KernelError("stream_shift: the stream and the row are float32")
+    if _delta_dtype(delta) != F32:
+        raise KernelError("stream_shift: a pending product is float32")
+    _check(lib, lib.mhb_stream_shift(_ptr(x), *_delta_args(delta), _ptr(table),
+                                     c_int(dtype_code(table.dtype) if table is not None else F32), _ptr(tokens),
+                                     c_float(scale), c_int(table.shape[0] if table is not None else 0), _ptr(row), c_int(T),
+                                     c_int(H), _stream()), "stream_shift")
+
+
+def _slot_state(state, n: int, what: str):
+    if state.dtype != torch.float32 or state.stride(-1) != 1 or state.shape[-1] < n:
+        raise KernelError(f"{what}: a slot holds {n} float32 numbers")
+    return _ptr(state), c_longlong(state.stride(0))
+
+
+def mingru_scan(proj, z0, x0, g0, bz, bx, state, ctx, out, *, writable=True):
+    """From columns of the float32 Product ``proj``: z = sigmoid(. + bz), u = . + bx, c = u + 1/2 where u >= 0 else
+    sigmoid(u); S <- (1 - z) S + z c per channel over ``state`` [slots, W]; out = S silu(g)."""
+    lib = build.load("selscan")
+    T, W = out.shape
+    p = proj.tensor
+    if p.dtype != torch.float32 or not out.is_contiguous():
+        raise KernelError("mingru_scan: the product is float32, the output contiguous")
+    _check(lib, lib.mhb_mingru_scan(*_parts_args(p, proj.nsplit, proj.split_stride), c_int(p.stride(-2)), c_int(z0), c_int(x0),
+                                    c_int(g0), _ptr(bz), _ptr(bx), *_slot_state(state, W, "mingru_scan"), *_seg_args(ctx),
+                                    _ptr(out), c_int(dtype_code(out.dtype)), c_int(T), c_int(len(ctx.segments)),
+                                    c_int(ctx.longest), c_int(W), c_int(1 if writable else 0), _stream()), "mingru_scan")
+
+
+SELECTIVE_STATES = 256      # states per channel the selective scan takes
+
+
+def selective_split(proj, rank: int, states: int, dt, bc):
+    """The product [dt: rank | B: states | C: states] apart: ``dt`` [T, >= rank] in its dtype (columns beyond the rank are
+    zero), ``bc`` float32 [T, 2 states]."""
+    lib = build.load("selscan")
+    p = proj.tensor
+    if p.dtype != torch.float32 or bc.dtype != torch.float32 or not bc.is_contiguous() or not dt.is_contiguous():
+        raise KernelError("selective_split: a float32 product, contiguous outputs")
+    _check(lib, lib.mhb_selective_split(*_parts_args(p, proj.nsplit, proj.split_stride), c_int(p.stride(-2)), c_int(rank),
+                                        c_int(states), _ptr(dt), c_int(dtype_code(dt.dtype)), c_int(dt.shape[1]), _ptr(bc),
+                                        c_int(dt.shape[0]), _stream()), "selective_split")
+
+
+def selective_scan(z, z0, dt, bc, b0, x, dt_bias, A2, D, state, ctx, out, *, dt_weight=None, rank=0, scale=1.0, writable=True):
+    """S <- exp(dt A) S + dt x B, y = S C + D x, out = y silu(z) * scale over ``state`` [slots, C N]; dt = softplus(. +
+    dt_bias).  ``z``, ``dt`` and ``bc`` are float32 Products (the gate's columns from z0, B and C from b0).  With
+    ``dt_weight`` [C, >= rank] the step's logits are that matrix times the first ``rank`` columns of ``dt`` (few tokens:
+    saves a product); else ``dt`` holds the logits [T, C].  ``A2`` [C, N]: A times log2(e)."""
+    lib = build.load("selscan")
+    T, C = out.shape
+    N = A2.shape[1]
+    if N > SELECTIVE_STATES:
+        raise KernelError(f"selective_scan: {N} states per channel (up to {SELECTIVE_STATES})")
+    for name, t in (("x", x), ("A", A2), ("D", D), ("dt's bias", dt_bias)):
+        if t.dtype != torch.float32 or not t.is_contiguous():
+            raise KernelError(f"selective_scan: {name} must be contiguous float32")
+    if dt_weight is not None and (dt_weight.dtype != out.dtype or dt_weight.stride(-1) != 1):
+        raise KernelError("selective_scan: dt's matrix has the output's dtype")
+    zt, bt = z.tensor[..., z0:], bc.tensor[..., b0:]
+    _check(lib, lib.mhb_selective_scan(
+        *_parts_args(zt, z.nsplit, z.split_stride), c_int(zt.stride(-2)),
+        *_parts_args(dt.tensor, dt.nsplit, dt.split_stride), c_int(dt.tensor.stride(-2)),
+        *_parts_args(bt, bc.nsplit, bc.split_stride), c_int(bt.stride(-2)), _ptr(x), _ptr(dt_weight), c_int(rank),
+        c_int(dt_weight.stride(0) if dt_weight is not None else 0), _ptr(dt_bias), _ptr(A2), _ptr(D),
+        *_slot_state(state, C * N, "selective_scan"), *_seg_args(ctx), _ptr(out), c_int(dtype_code(out.dtype)), c_float(scale),
+        c_int(T), c_int(len(ctx.segments)), c_int(C), c_int(N), c_int(1 if writable else 0), _stream()), "selective_scan")

@@ -1,2 +1,2 @@
-from . import dotivik, koronex, qwen2, rizovik, tudasun  # noqa: F401  (register Dotivik, Koronex, Qwen2ForCausalLM, Rizovik and Tudasun)
+from . import dotivik, koronex, qwen2, rizovik, tudasun, zetenex  # noqa: F401  (each registers its architecture)
 from .decoder import DecoderModel

@@ -43,6 +43,14 @@ class DecoderModel:
                         f"{mine} vs {theirs}"
                     )
                 self.entry_cache.append(owner)
+        # memory beside that (StateNeed beside pages, ...): run entry -> {name: cache entry index}; never shared
+        self.entry_sides: list[dict[str, int]] = []
+        for e in spec.order:
+            sides = {}
+            for name, need in self.blocks[e.layer].side_needs().items():
+                sides[name] = len(self.cache_needs)
+                self.cache_needs.append(need)
+            self.entry_sides.append(sides)
         self.loaded = False
 
     # ---- parameters --------------------------------------------------------------------------
@@ -77,14 +85,17 @@ class DecoderModel:
     def finish_loading(self):
         if getattr(self.head, "tied", False):
             self.head.tie(self.embedding)
+        for part in self.shared.values():
+            if hasattr(part, "tie"):           # a part that reads the embedding table again
+                part.tie(self.embedding)
         self.loaded = True
 
     def weight_bytes(self) -> int:
         seen, total = set(), 0
         parts = [p for _, p in self.named_parts()]
         for part in parts:
-            for v in vars(part).values():
-                if isinstance(v, torch.Tensor) and v.data_ptr() not in seen:
+            for v in part.tensors():
+                if v.data_ptr() not in seen:
                     seen.add(v.data_ptr())
                     total += v.numel() * v.element_size()
         return total
@@ -111,8 +122,9 @@ class DecoderModel:
             view = caches[i]
             block = self.blocks[entry.layer]
             if entry.before is not None:       # a part of the model as a whole transforms the stream first
-                x, pending = self.shared[entry.before].forward_stream(x, pending, ctx)
+                x, pending = self.shared[entry.before].forward_stream(x, pending, ctx, entry.turn)
             pending = block.forward(x, pending, ctx, view)
+            x = ctx.extras.pop("stream", x)        # a block may have moved the stream to another buffer
             if not block.keeps_copy:
                 ctx.extras.pop("x_copy", None)     # whoever changed the stream did not keep its copy in step
             if observer is not None:

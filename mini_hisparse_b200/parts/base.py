@@ -21,7 +21,7 @@ Interfaces, in short:
 """
 from __future__ import annotations
 
-from dataclasses import dataclass, field
+from dataclasses import dataclass, field, replace
 from typing import Any
 
 import numpy as np
@@ -204,6 +204,12 @@ class CacheView:
     storage: torch.Tensor | None    # pages: [pages, 2, nkv, P, d]; state: [max_requests, *shape]
     page_size: int = 0
     meta: dict = field(default_factory=dict)   # device views of the group's per-step arrays
+    sides: dict = field(default_factory=dict)  # name -> CacheView of the memory asked for beside it (side_needs)
+
+    def narrow(self, prefix: str) -> "CacheView":
+        """The same view for a part inside the one it was made for: only the side memory whose names
+        start with ``prefix``, under the rest of those names."""
+        return replace(self, sides={k[len(prefix):]: v for k, v in self.sides.items() if k.startswith(prefix)})
 
 
 @dataclass
@@ -217,7 +223,13 @@ class StepContext:
     tok_seg: torch.Tensor           # [T] int32: segment of each token
     seg_slot: torch.Tensor          # [S] int32: state slot of each segment
     status: torch.Tensor            # [1] int32 error bits set by kernels
+    seg_offset: torch.Tensor | None = None   # [S + 1] int32: first token of each segment, and T
     extras: dict = field(default_factory=dict)
+
+    @property
+    def longest(self) -> int:
+        """Tokens of the step's longest segment (1 in a step of single tokens)."""
+        return max((s.count for s in self.segments), default=0)
 
 
 # ---------------------------------------------------------------------------------------
@@ -241,11 +253,15 @@ class Part:
             setattr(self, k.replace(".", "_"), v)
 
     def nbytes(self) -> int:
-        total = 0
+        return sum(v.numel() * v.element_size() for v in self.tensors())
+
+    def tensors(self):
+        """Every tensor the part holds, those of parts inside it included."""
         for v in vars(self).values():
             if isinstance(v, torch.Tensor):
-                total += v.numel() * v.element_size()
-        return total
+                yield v
+            elif isinstance(v, Mixer):
+                yield from v.tensors()
 
 
 class StepPlanner:
@@ -292,6 +308,15 @@ class Mixer(Part):
     def cache_need(self) -> CacheNeed | None:
         return None
 
+    def side_needs(self) -> dict[str, CacheNeed]:
+        """Per-request memory beside cache_need(), by name (a mixer that keeps pages AND a recurrent state):
+        forward() finds its views in ``cache.sides``.  Every run entry has its own."""
+        return {}
+
+    def side_user(self, name: str):
+        """Who brings the plan for that memory's group (an object with plan_key() and planner()), or None."""
+        return None
+
     def plan_key(self):
         """Mixers of one page group with equal keys share a planner (None: no plan needed)."""
         return None
@@ -324,7 +349,9 @@ class Block:
     in ``parts()`` (role -> part, the roles of its LayerSpec), and names the ONE part that owns
     per-request memory as ``self.mixer`` (or overrides the three methods below).
     ``forward(x, pending, ctx, cache) -> pending``: x is the float32 residual [T, H]; ``pending``
-    is the previous block's last output, not yet added to x (None for the first block).
+    is the previous block's last output, not yet added to x (None for the first block).  A block
+    whose kernels write the stream to another buffer than they read it from leaves the new one as
+    ctx.extras["stream"] (stream_other() gives the buffer).
     """
 
     mixer: "Mixer | None" = None
@@ -333,6 +360,12 @@ class Block:
 
     def parts(self) -> dict[str, Part]:
         raise NotImplementedError
+
+    @staticmethod
+    def stream_other(x: torch.Tensor, ctx: StepContext) -> torch.Tensor:
+        """The buffer of a pair that does not hold the stream ``x`` now."""
+        a = ctx.ws.get("residual", tuple(x.shape), torch.float32)
+        return a if a.data_ptr() != x.data_ptr() else ctx.ws.get("residual_other", tuple(x.shape), torch.float32)
 
     def kernel_modules(self) -> tuple[str, ...]:
         """Kernel libraries the arrangement itself launches, beyond those of its parts."""
@@ -343,6 +376,14 @@ class Block:
 
     def cache_need(self) -> CacheNeed | None:
         return self.mixer.cache_need() if self.mixer is not None else None
+
+    def side_needs(self) -> dict[str, CacheNeed]:
+        """Memory beside cache_need(): the mixer's under "mixer.<name>"; an arrangement that keeps something
+        of its own adds it."""
+        return {"mixer." + k: v for k, v in self.mixer.side_needs().items()} if self.mixer is not None else {}
+
+    def side_user(self, name: str):
+        return self.mixer.side_user(name[len("mixer."):]) if name.startswith("mixer.") else None
 
     def plan_key(self):
         return self.mixer.plan_key() if self.mixer is not None else None

@@ -5,8 +5,8 @@ import torch
 
 from ..kernels import api as K
 from .base import Block, CacheView, Product, StepContext
-from .registry import FEED_FORWARDS, GATES, MIXERS, NORMS, register_block
-from .spec import LayerSpec
+from .registry import FEED_FORWARDS, GATES, INPUT_CONVS, MIXERS, NORMS, register_block
+from .spec import LayerSpec, StateNeed
 
 
 @register_block("pre_norm")
@@ -232,3 +232,59 @@ class SandwichBlock(Block):
         if self.side is not None:
             self.side.forward_into(x, x if copy is None else copy, ctx, keep_copy=False)
         return None
+
+
+@register_block("pre_norm_conv")
+class PreNormConvBlock(Block):
+    """Pre-norm with a short causal convolution over time in front of each sublayer:
+
+        h = norm1(x);  x <- x + mixer(h + conv1(h));   h = norm2(x);  x <- x + ff(h + conv2(h))   (if there is one)
+
+    Roles: "mixer_norm", "mixer_conv", "mixer", and optionally "ff_norm", "ff_conv", "feed_forward".  A sequence's last
+    taps - 1 inputs of both convolutions are side memory "input_conv" [1 or 2, taps - 1, width].  Residual additions are
+    folded into the norm that follows; with a norm that works element by element (forward_conv), the norm and the
+    convolution are one kernel, which moves the stream to another buffer.
+    """
+
+    def __init__(self, spec: LayerSpec, rt):
+        self.spec = spec
+        self.mixer_norm = NORMS.build(spec.part("mixer_norm"), rt=rt)
+        self.mixer_conv = INPUT_CONVS.build(spec.part("mixer_conv"), rt=rt)
+        self.mixer = MIXERS.build(spec.part("mixer"), rt=rt)
+        self.ff_norm = self.ff_conv = self.feed_forward = None
+        if spec.has("feed_forward"):
+            self.ff_norm = NORMS.build(spec.part("ff_norm"), rt=rt)
+            self.ff_conv = INPUT_CONVS.build(spec.part("ff_conv"), rt=rt)
+            self.feed_forward = FEED_FORWARDS.build(spec.part("feed_forward"), rt=rt)
+            if self.ff_conv.kept_shape != self.mixer_conv.kept_shape:
+                raise ValueError("a layer's two input convolutions have one shape")
+
+    def parts(self):
+        out = {"mixer_norm": self.mixer_norm, "mixer_conv": self.mixer_conv, "mixer": self.mixer}
+        if self.feed_forward is not None:
+            out.update(ff_norm=self.ff_norm, ff_conv=self.ff_conv, feed_forward=self.feed_forward)
+        return out
+
+    def side_needs(self):
+        out = super().side_needs()
+        rows, width = self.mixer_conv.kept_shape
+        if rows:
+            out["input_conv"] = StateNeed(shape=(1 if self.feed_forward is None else 2, rows, width), dtype="float32")
+        return out
+
+    def _input(self, x, norm, conv, which: int, delta, ctx: StepContext, cache: CacheView):
+        """(the stream's buffer, norm and convolution of the stream with ``delta`` added)."""
+        view = cache.sides.get("input_conv")
+        kept = view.storage[:, which] if view is not None else None
+        if hasattr(norm, "forward_conv"):
+            return norm.forward_conv(x, ctx, conv, kept, delta=delta, other=self.stream_other(x, ctx))
+        return x, conv.forward(norm.forward(x, ctx, delta=delta), ctx, kept)
+
+    def forward(self, x, pending: Product | None, ctx: StepContext, cache: CacheView | None) -> Product:
+        x, h = self._input(x, self.mixer_norm, self.mixer_conv, 0, pending, ctx, cache)
+        out = self.mixer.forward(h, ctx, cache.narrow("mixer."))
+        if self.feed_forward is not None:
+            x, h = self._input(x, self.ff_norm, self.ff_conv, 1, out, ctx, cache)
+            out = self.feed_forward.forward(h, ctx)
+        ctx.extras["stream"] = x
+        return out

@@ -85,12 +85,47 @@ class StreamInput(Part):
     def load(self, tensors):
         self.weight = tensors[self.weight_name].contiguous()
 
-    def forward_stream(self, x, pending: Product | None, ctx: StepContext):
+    def forward_stream(self, x, pending: Product | None, ctx: StepContext, turn: int = 0):
         cat = ctx.extras.get(self.buffer)
         if cat is None:
             raise RuntimeError(f"the embedding did not keep its output in {self.buffer!r}")
         K.stream_pack(x, cat, 0, delta=pending, delta2=pending.also if pending is not None else None, zero=True)
         return x, ctx.rt.linear(cat, self.weight, ctx.ws, "stream_in", out_dtype=torch.float32)
+
+
+@EMBEDDINGS.register("pass_input")
+class PassInput(Part):
+    """A part of the model as a whole that opens every pass over repeated layers:  x <- x + x0 (not before the
+    first pass), then x <- x + step[turn], with x0 the embedding output (the table's row times the embedding's
+    scale, gathered again rather than kept) and ``step`` [times, width] one stored vector per pass.  Everything
+    pending is added in the same kernel, in float32.  Parameters: width, times, weight_name."""
+
+    def __init__(self, spec: PartSpec, rt=None):
+        super().__init__(spec, rt)
+        self.width, self.times = int(spec["width"]), int(spec["times"])
+        self.weight_name = spec.get("weight_name", "step")
+        self.step = None
+        self._embedding = None
+
+    def kernel_modules(self):
+        return ("timeconv",)
+
+    def parameters(self):
+        return {self.weight_name: ParamSpec((self.times, self.width), role="vector", init=("normal", 0.0, 0.1))}
+
+    def load(self, tensors):
+        self.step = tensors[self.weight_name].float().contiguous()
+
+    def tie(self, embedding: TokenEmbedding):
+        self._embedding = embedding
+
+    def forward_stream(self, x, pending: Product | None, ctx: StepContext, turn: int = 0):
+        if pending is not None:
+            pending = pending.settle_also(x)
+        e = self._embedding
+        K.stream_shift(x, self.step[turn], delta=pending, table=e.weight if turn else None, tokens=ctx.tokens,
+                       scale=e.scale)
+        return x, None
 
 
 @EMBEDDINGS.register("token_table")

@@ -100,3 +100,53 @@ class LayerNorm(Norm):
             second = second.settle_also(x)
         K.add_layernorm(x, self.weight, self.eps, out, delta=delta, delta2=second, rows=rows)
         return out
+
+
+@register_norm("dyt")
+class DynamicTanh(Norm):
+    """y = tanh(alpha x) * weight + shift with one stored number alpha: a bounded squashing in place of a norm, which
+    takes no mean and no variance.  Computed in float32 from the float32 residual; pending products are added first.
+    Since it works element by element, a convolution over time that follows it runs in the same kernel (forward_conv).
+    Parameters: width, weight_name (default "weight").  Tensors: the weight, and beside it "alpha" (a scalar) and "b"."""
+
+    def __init__(self, spec: PartSpec, rt=None):
+        super().__init__(spec, rt)
+        self.width = int(spec["width"])
+        self.weight_name = spec.get("weight_name", "weight")
+        self.weight = self.alpha = self.shift = None
+
+    def kernel_modules(self):
+        return ("timeconv",)
+
+    def parameters(self):
+        return {self.weight_name: ParamSpec((self.width,), role="vector", init=("normal", 1.0, 0.1)),
+                "b": ParamSpec((self.width,), role="vector", init=("normal", 0.0, 0.1)),
+                "alpha": ParamSpec((), role="vector", init=("normal", 0.6, 0.1))}
+
+    def load(self, tensors):
+        self.weight, self.shift = tensors[self.weight_name].contiguous(), tensors["b"].contiguous()
+        self.alpha = tensors["alpha"].reshape(1).contiguous()
+
+    def _two(self, delta: Product | None, x):
+        """At most two products for the kernel; more are settled into the stream first."""
+        second = delta.also if delta is not None else None
+        if second is not None and second.also is not None:
+            second = second.settle_also(x)
+        return delta, second
+
+    def forward(self, x, ctx: StepContext, delta: Product | None = None, rows=None, name="h"):
+        R = x.shape[0] if rows is None else rows.shape[0]
+        out = ctx.ws.get(name, (R, self.width), ctx.rt.dtype)
+        delta, second = self._two(delta, x)
+        K.dyt_rows(x, self.alpha, self.weight, self.shift, out, delta=delta, delta2=second, rows=rows)
+        return out
+
+    def forward_conv(self, x, ctx: StepContext, conv, kept, delta: Product | None = None, other=None, name="h",
+                     writable=True):
+        """The norm and h <- h + conv(h) in one kernel.  The sum x + delta goes to ``other`` (a second buffer of the
+        stream's shape: a token's inputs are read by its successors too); returns (the stream's buffer now, the rows)."""
+        out = ctx.ws.get(name, tuple(x.shape), ctx.rt.dtype)
+        delta, second = self._two(delta, x)
+        K.stream_conv(x, self.alpha, self.weight, self.shift, conv.filters, kept, ctx, out, delta=delta, delta2=second,
+                      x_out=other if delta is not None else None, writable=writable)
+        return (x if delta is None else other), out

@@ -50,6 +50,7 @@ BLOCKS = Registry("block arrangement")
 EMBEDDINGS = Registry("embedding")
 HEADS = Registry("output head")
 GATES = Registry("gate")
+INPUT_CONVS = Registry("input convolution")
 
 register_mixer: Callable = MIXERS.register
 register_feed_forward: Callable = FEED_FORWARDS.register
@@ -57,3 +58,4 @@ register_norm: Callable = NORMS.register
 register_position: Callable = POSITIONS.register
 register_block: Callable = BLOCKS.register
 register_gate: Callable = GATES.register
+register_input_conv: Callable = INPUT_CONVS.register

@@ -117,6 +117,13 @@ class SinkAttention(Mixer):
         g0 = self.qw + (self.kw + self.vw if self.own_kv else 0)
         gate = dict(gate=(p[0] if proj.nsplit > 1 else p)[:, g0:], gate_nsplit=proj.nsplit,
                     gate_split_stride=proj.split_stride)
+        attn = self._attend(q, gate, ctx, cache, sink=self.sink)
+        return rt.linear(attn, self.o_weight, ws, "mix_out", out_dtype=torch.float32)
+
+    def _attend(self, q, gate: dict, ctx: StepContext, cache: CacheView, sink=None) -> torch.Tensor:
+        """The plan's items over the cache, the merge of key splits and the gate: [T, q_heads * vdim] in the compute dtype."""
+        rt, ws, T = ctx.rt, ctx.ws, q.shape[0]
+        meta = cache.meta
         attn = ws.get("sa_attn", (T, self.ow), rt.dtype)
         part_rows = max(1, meta["part_rows_cap"])
         part_acc = ws.get("attn_part_acc", (part_rows, self.nq, self.dv), torch.float32)
@@ -128,14 +135,14 @@ class SinkAttention(Mixer):
             args = (q, cache.storage, attn, part_acc, part_ml)
             tail = (ctx.positions, meta["block_table"], meta["tok_part_row"])
             common = dict(nq=self.nq, nkv=self.nkv, d=self.dk, dv=self.dv, page_size=cache.page_size,
-                          window=self.window or 0, scale=self.scale, sink=self.sink, **gate)
+                          window=self.window or 0, scale=self.scale, sink=sink, **gate)
             if n_small:          # decoded tokens and short portions: 16-row tiles, key splits merged by the last CTA
                 chunks = -(-(self.nq // self.nkv) // ROW_TILE)
                 counters = ws.get_zeroed("attn_counters", (T * self.nkv * chunks,), torch.int32)
                 if family == "tc":      # TMA-fed tiles (keys and values of one width, pages that divide 64)
                     K.attention_tma_ext(*args, meta["items"], n_small, 16, *tail, nq=self.nq, nkv=self.nkv, d=self.dk,
                                         page_size=cache.page_size, window=self.window or 0, scale=self.scale,
-                                        sink=self.sink, **gate, tok_nsplit=meta["tok_nsplit"], counters=counters,
+                                        sink=sink, **gate, tok_nsplit=meta["tok_nsplit"], counters=counters,
                                         status=ctx.status)
                 else:
                     K.attention_mma_ext(*args, meta["items"], n_small, 16, *tail, **common,
@@ -145,19 +152,19 @@ class SinkAttention(Mixer):
                 K.attention_tc_ext(q, cache.storage, attn, big_items, n_big, ctx.positions, meta["block_table"],
                                    nq=self.nq, nkv=self.nkv, d=self.dk, page_size=cache.page_size,
                                    window=self.window or 0, scale=self.scale, status=ctx.status, part_acc=part_acc,
-                                   part_ml=part_ml, tok_part_row=meta["tok_part_row"], sink=self.sink, **gate)
+                                   part_ml=part_ml, tok_part_row=meta["tok_part_row"], sink=sink, **gate)
                 if meta.get("big_split"):
                     K.attention_combine(part_acc, part_ml, meta["tok_part_row"], meta["tok_nsplit"], attn,
                                         nq=self.nq, d=self.dv, **gate)
             elif n_big:          # long portions: 64-row tiles
                 K.attention_mma_ext(*args, big_items, n_big, 64, *tail, **common)
-            return rt.linear(attn, self.o_weight, ws, "mix_out", out_dtype=torch.float32)
+            return attn
         if n:
             K.attention_simt(q, cache.storage, attn, part_acc, part_ml, meta["items"], n, n, ctx.positions,
                              meta["block_table"], meta["tok_part_row"], nq=self.nq, nkv=self.nkv, d=self.dk,
                              dv=self.dv, page_size=cache.page_size, window=self.window or 0, scale=self.scale,
-                             sink=self.sink, **gate)
+                             sink=sink, **gate)
         if meta["any_split"]:
             K.attention_combine(part_acc, part_ml, meta["tok_part_row"], meta["tok_nsplit"], attn, nq=self.nq,
                                 d=self.dv, **gate)
-        return rt.linear(attn, self.o_weight, ws, "mix_out", out_dtype=torch.float32)
+        return attn

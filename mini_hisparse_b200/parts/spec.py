@@ -115,11 +115,14 @@ class RunEntry:
     index of an EARLIER entry of the run order whose cache this entry only reads.
     ``before``: the key of a part of the model as a whole (ModelSpec.shared) that transforms the
     residual stream right before this entry runs (the input of a pass over repeated layers).
+    ``turn``: which of its uses of that part this is (the number of the pass), for a part that does
+    not do the same every time.
     """
 
     layer: int
     cache_of: int | None = None
     before: str | None = None
+    turn: int = 0
 
 
 @dataclass(frozen=True)
