@@ -156,11 +156,15 @@ template <> __device__ __forceinline__ void store_out<__nv_bfloat16>(__nv_bfloat
 
 // EPI 1 and 3 are the gated epilogues: act(gate) * up with act = silu (1) or the tanh form of gelu (3).
 __host__ __device__ constexpr bool is_glu(int epi) { return epi == 1 || epi == 3; }
+// EPI 4 applies the tanh form of gelu to every element (no gate).
+__device__ __forceinline__ float gelu_tanh(float g) {
+    const float c = 0.7978845608028654f;      // sqrt(2 / pi)
+    return 0.5f * g * (1.f + tanhf(c * (g + 0.044715f * g * g * g)));
+}
 template <int EPI>
 __device__ __forceinline__ float glu_mul(float g, float u) {
     if constexpr (EPI == 3) {
-        const float c = 0.7978845608028654f;      // sqrt(2 / pi)
-        return 0.5f * g * (1.f + tanhf(c * (g + 0.044715f * g * g * g))) * u;
+        return gelu_tanh(g) * u;
     } else {
         return g / (1.f + expf(-g)) * u;
     }
@@ -431,8 +435,12 @@ struct QkvRopeArgs {
 // columns c0.. of the tile whose first column is rb0.
 template <typename OT, int EPI>
 __device__ __forceinline__ void emit_unit(OT* __restrict__ C, long long ldc, int Ra, int Rb, int ra, int rb0, int c0,
-                                          const uint32_t (&r)[16], const uint32_t (&r2)[16]) {
+                                          uint32_t (&r)[16], const uint32_t (&r2)[16]) {
     if (ra >= Ra) return;
+    if constexpr (EPI == 4) {
+#pragma unroll
+        for (int x = 0; x < 16; ++x) r[x] = __float_as_uint(gelu_tanh(__uint_as_float(r[x])));
+    }
     if constexpr (is_glu(EPI)) {
         OT* row = C + (size_t)ra * ldc + (rb0 + c0) / 2;
         float v[16];
@@ -1512,4 +1520,15 @@ MHB_EXPORT int mhb_gemm_tc_glu(const void* X, const void* W, void* C, int c_dtyp
     if (act == 0) return gemm_tc_glu<1>(X, W, C, c_dtype, M, I, K, lda, ldw, ldc, swap, bn, partials, flags, status, stream);
     if (act == 1) return gemm_tc_glu<3>(X, W, C, c_dtype, M, I, K, lda, ldw, ldc, swap, bn, partials, flags, status, stream);
     return fail("gemm_tc_glu: unknown activation %d", act);
+}
+
+// C[M, N] = act(X W^T), bfloat16 out, the activation (1 = the tanh form of gelu) taken in float32 on the accumulators in
+// the persistent product's epilogue (more than 64 tokens).
+MHB_EXPORT int mhb_gemm_tc_act(const void* X, const void* W, void* C, int M, int N, int K, long long lda, long long ldw,
+                               long long ldc, float* partials, int* flags, int* status, int act, cudaStream_t stream) {
+    if (M <= 0 || N <= 0) return 0;
+    if (act != 1) return fail("gemm_tc_act: unknown activation %d", act);
+    if (K <= 0 || K % 8 || lda % 8 || ldw % 8) return fail("gemm_tc: K, lda and ldw must be multiples of 8 (K %d, lda %lld, ldw %lld)", K, lda, ldw);
+    if (((uintptr_t)X & 15) || ((uintptr_t)W & 15)) return fail("gemm_tc: operands must be 16-byte aligned");
+    return launch_persistent<__nv_bfloat16, 4>(X, W, C, M, N, K, lda, ldw, ldc, partials, flags, status, stream);
 }

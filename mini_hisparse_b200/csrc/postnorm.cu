@@ -252,7 +252,9 @@ __global__ void qknorm_rope_append_kernel(const float* __restrict__ qkv, int nsp
     if (v_eps > 0.f)
         for (int i = threadIdx.x; i < vw; i += blockDim.x) vs[i] = load_parts(qkv, base + qw + kw + i, nsplit, split_stride);
     if (per_head) {
-        // one norm per head over its dk elements, the weight [dk] shared by the heads: a warp per head
+        // one norm per head over its dk elements, the weight [dk] shared by the heads: a warp per head; and a temperature
+        // that grows with the position, on q alone: 1 + coef ln(floor((pos + 1) / every) + 1)
+        const float temp = temp_coef != 0.f ? 1.f + temp_coef * log1pf((float)floor((double)(pos + 1) / temp_every)) : 1.f;
         __syncthreads();
         const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
         for (int head = warp; head < (qw + kw) / dk; head += nwarps) {
@@ -261,9 +263,7 @@ __global__ void qknorm_rope_append_kernel(const float* __restrict__ qkv, int nsp
             float ss = 0.f;
             for (int e = lane; e < dk; e += 32) ss += row[e] * row[e];
             const float r = 1.f / sqrtf(warp_sum(ss) / (float)dk + eps);
-            // a temperature that grows with the position, on q alone: 1 + coef ln(floor((pos + 1) / every) + 1)
-            const float f = head < nq && temp_coef != 0.f
-                                ? 1.f + temp_coef * log1pf((float)floor((double)(pos + 1) / temp_every)) : 1.f;
+            const float f = head < nq ? temp : 1.f;
             for (int e = lane; e < dk; e += 32) row[e] = row[e] * r * (w ? w[e] : 1.f) * f;
         }
     } else {

@@ -92,7 +92,7 @@ template <int VEC> __device__ __forceinline__ void add_parts(const float* p, int
     }
 }
 
-__device__ __forceinline__ float silu(float z) { return z / (1.f + expf(-z)); }
+__device__ __forceinline__ float silu(float z) { return __fdividef(z, 1.f + expf(-z)); }
 
 // the raw input of one token: the stream with everything pending, or the rows themselves
 template <int MODE, typename IT, int VEC>
@@ -260,21 +260,30 @@ __global__ void dyt_rows_kernel(float* __restrict__ x, Delta d1, Delta d2, const
 }
 
 // ---- x <- x + d (+ table[token] scale) + row ---------------------------------------------------------
-template <typename WT>
+template <typename WT, int VEC>
 __global__ void stream_shift_kernel(float* __restrict__ x, Delta d, const WT* __restrict__ table, const int* __restrict__ tokens,
-                                    float scale, int vocab, const float* __restrict__ row, int H) {
+                                    float scale, int vocab, const float* __restrict__ row, size_t n, int H) {
     pdl_launch_dependents();
     pdl_wait();
-    const size_t t = blockIdx.y;
-    const int i = blockIdx.x * blockDim.x + threadIdx.x;
-    if (i >= H) return;
-    float v[1] = {x[t * H + i]};
-    if (d.p) add_parts<1>(d.p + t * H + i, d.nsplit, d.stride, v);
+    const size_t at = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * VEC;
+    if (at >= n) return;
+    const size_t t = at / H;
+    const int i = (int)(at - t * H);
+    float v[VEC], e[VEC], r[VEC];
+    load_f<VEC>(x + at, v);
+    load_f<VEC>(row + i, r);
+    if (d.p) add_parts<VEC>(d.p + at, d.nsplit, d.stride, v);
     if (table) {
         const int tok = tokens[t];                    // an id outside the table gave zeros (and a status bit) in the embedding
-        if (tok >= 0 && tok < vocab) v[0] += to_float(table[(size_t)tok * H + i]) * scale;
+        if (tok >= 0 && tok < vocab) {
+            load_f<VEC>(table + (size_t)tok * H + i, e);
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) v[j] += e[j] * scale;
+        }
     }
-    x[t * H + i] = v[0] + row[i];
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) v[j] += r[j];
+    store_f<VEC>(x + at, v);
 }
 }  // namespace
 
@@ -343,13 +352,14 @@ MHB_EXPORT int mhb_stream_shift(float* x, const float* d, int nd, long long sd, 
                                 const int* tokens, float scale, int vocab, const float* row, int T, int H,
                                 cudaStream_t stream) {
     if (T <= 0) return 0;
-    const int threads = 128;
-    const int blocks = (H + threads - 1) / threads;
-    for (int t = 0; t < T; t += 65535) {
-        const int n = T - t < 65535 ? T - t : 65535;
-        MHB_DISPATCH_DTYPE(table_dtype, WT,
-            launch_kernel(stream_shift_kernel<WT>, dim3(blocks, n), dim3(threads), 0, stream, x + (size_t)t * H,
-                          Delta{d ? d + (size_t)t * H : nullptr, nd, (size_t)sd}, (const WT*)table, tokens + t, scale, vocab, row, H));
-    }
+    const size_t n = (size_t)T * H;
+    const Delta delta{d, nd, (size_t)sd};
+    const bool vec = H % 4 == 0 && aligned16(x) && aligned16(d) && sd % 4 == 0 && aligned16(table) && aligned16(row);
+    const int per = vec ? 4 : 1, threads = 128;
+    const unsigned blocks = (unsigned)((n / per + threads - 1) / threads);
+    MHB_DISPATCH_DTYPE(table_dtype, WT, {
+        if (vec) launch_kernel(stream_shift_kernel<WT, 4>, dim3(blocks), dim3(threads), 0, stream, x, delta, (const WT*)table, tokens, scale, vocab, row, n, H);
+        else launch_kernel(stream_shift_kernel<WT, 1>, dim3(blocks), dim3(threads), 0, stream, x, delta, (const WT*)table, tokens, scale, vocab, row, n, H);
+    });
     return check_launch("stream_shift");
 }

@@ -415,6 +415,26 @@ def gemm_tc_glu(a, w, out, act: str, *, swap: bool, bn: int, status=None, scratc
         "gemm_tc_glu")
 
 
+PRODUCT_ACTS = ("gelu_tanh",)       # activations that the tensor-core product's epilogue takes without a gate
+
+
+def gemm_tc_act(a, w, out, act: str, *, status=None, scratch=None):
+    """out[M, N] = act(a w^T) in bfloat16, the activation taken in float32 on the accumulators in the persistent
+    product's epilogue (more than 64 tokens)."""
+    lib = build.load("gemm_tc")
+    M, K = a.shape
+    N = w.shape[0]
+    if a.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or out.dtype != torch.bfloat16:
+        raise KernelError("gemm_tc_act: operands and output must be bfloat16")
+    if w.shape[1] != K or tuple(out.shape) != (M, N) or act not in PRODUCT_ACTS:
+        raise KernelError(f"gemm_tc_act: a is [{M},{K}], w {list(w.shape)}, out {list(out.shape)}, activation {act!r}")
+    if a.stride(1) != 1 or w.stride(1) != 1 or out.stride(1) != 1:
+        raise KernelError("gemm_tc_act: the last dimension must be contiguous")
+    _check(lib, lib.mhb_gemm_tc_act(
+        _ptr(a), _ptr(w), _ptr(out), c_int(M), c_int(N), c_int(K), c_longlong(a.stride(0)), c_longlong(w.stride(0)),
+        c_longlong(out.stride(0)), *_scratch_ptrs(scratch), _ptr(status), c_int(GLU_ACTS[act]), _stream()), "gemm_tc_act")
+
+
 def rope_table(positions, inv_freq, table):
     """table[t] = cos of token t's rotation angles, then their sin (float32, [T, 2 * angles]), for the
     q/k/v product's rotating epilogue."""

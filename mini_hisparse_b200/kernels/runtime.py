@@ -95,6 +95,24 @@ class BFloat16Runtime(Runtime):
             return out
         return super().linear_glu(x, weight, block, activation, ws, name)
 
+    def linear_act(self, x, weight, activation: str, ws: Workspace, name: str) -> torch.Tensor:
+        """Many tokens: the activation rides in the persistent product's epilogue, if it is one of those built in, so the
+        float32 matrix is never written; else the product is followed by the activation kernel."""
+        M, N = x.shape[0], weight.shape[0]
+        if (activation in K.PRODUCT_ACTS and M > 64 and 2 * -(-M // 128) * -(-N // 256) >= self.sm_count
+                and self._tc_takes(x, weight)):
+            out = ws.get(name, (M, N), self.dtype)
+            K.gemm_tc_act(x, weight, out, activation, status=self.status, scratch=self.scratch())
+            return out
+        return super().linear_act(x, weight, activation, ws, name)
+
+    @staticmethod
+    def _tc_takes(x, weight) -> bool:
+        """The operands' dtypes, widths, strides and addresses are those of the tensor-core product."""
+        return (x.dtype == torch.bfloat16 and weight.dtype == torch.bfloat16 and x.shape[1] % 8 == 0
+                and x.stride(0) % 8 == 0 and weight.stride(0) % 8 == 0
+                and x.data_ptr() % 16 == 0 and weight.data_ptr() % 16 == 0)
+
     def qkv_rope_append(self, x, weight, bias, ctx, position, block_table, q_out, cache_storage, *,
                         nq, nkv, d, page_size, write_kv) -> bool:
         """More than 64 tokens and head size 64 or 128: the persistent product's epilogue rotates and
@@ -127,10 +145,7 @@ class BFloat16Runtime(Runtime):
         M, Kd = x.shape
         N = weight.shape[0]
         out_dtype = out_dtype or self.dtype
-        tc_ok = (x.dtype == torch.bfloat16 and weight.dtype == torch.bfloat16 and bias is None
-                 and Kd % 8 == 0 and x.stride(0) % 8 == 0 and weight.stride(0) % 8 == 0
-                 and x.data_ptr() % 16 == 0 and weight.data_ptr() % 16 == 0)
-        if not tc_ok:
+        if bias is not None or not self._tc_takes(x, weight):
             out = ws.get(name, (M, N), out_dtype)
             K.gemm_simt(x, weight, out, bias=bias)
             return Product(out)

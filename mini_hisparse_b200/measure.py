@@ -484,6 +484,26 @@ def rizovik_shape(width: int, heads: int, kv_heads: int, head_dim: int, ff: int,
     return dict(architecture="Rizovik", vocab=vocab, width=width, norm=dict(eps=1e-6), residual_mult=0.5, layers=out)
 
 
+def zetenex_shape(width: int, heads: int, kv_heads: int, head_dim: int, ff: int, layers: int, vocab: int) -> dict:
+    """A Zetenex config.json of a real model's sizes with ``layers`` layer RUNS: groups of three layers (attention beside a
+    selective scan, two minGRU layers), of which two in the middle run twice.  The attention side has ``heads`` heads, the
+    scan ``width`` channels of 16 states with a step of rank width / 16 and four taps; minGRU layers are ``width`` wide;
+    every layer has a plain feed-forward ``ff`` wide."""
+    par = dict(left=dict(heads=heads, kv_heads=kv_heads, dim=head_dim, vdim=head_dim, scale=head_dim ** -0.5,
+                         q_temp=dict(coef=0.1, every=1024)), left_scale=0.7,
+               right=dict(inner=width, state=16, dt_rank=width // 16, conv=4), right_scale=0.7)
+    repeat = 2 if layers >= 4 else 0
+    stored = layers - repeat
+    out = [dict(type="mingru" if i % 3 else "parallel", mixer=dict(width=width) if i % 3 else par,
+                mlp=dict(kind="dense", ff=ff)) for i in range(stored)]
+    shape = dict(architecture="Zetenex", vocab=vocab, width=width, norm=dict(eps=1e-5), canon=dict(taps=4),
+                 embedding=dict(scale=float(width) ** 0.5), layers=out)
+    if repeat:
+        start = (stored - repeat) // 2
+        shape["loop"] = dict(start=start, stop=start + repeat, times=2)
+    return shape
+
+
 def qwen2_shape(width: int, heads: int, kv_heads: int, head_dim: int, ff: int, layers: int, vocab: int) -> dict:
     return dict(architectures=["Qwen2ForCausalLM"], model_type="qwen2", vocab_size=vocab, hidden_size=width,
                 intermediate_size=ff, num_hidden_layers=layers, num_attention_heads=heads,
@@ -497,7 +517,7 @@ class KernelTimes:
 
     SKIP = {"stream_scope", "dtype_code", "stream_k_scratch", "gemm_tc_wait_limit", "KernelError",
             "attention_decode_supports", "attention_tma_supports", "gemm_tc_qkv_rope_supports",
-            "attention_decode_max_clusters", "lightning_chunk_smem", "attention_mma_ext_supports",
+            "attention_decode_max_clusters", "lightning_chunk_smem", "c_double", "attention_mma_ext_supports",
             "lightning_chunked_tc_supports"}
 
     def __enter__(self):
@@ -660,17 +680,19 @@ COMPARE_SIZES = {
 
 
 DESIGN_SHAPES = {"koronex": koronex_shape, "dotivik": dotivik_shape, "tudasun": tudasun_shape, "rizovik": rizovik_shape,
-                 "qwen2": qwen2_shape}
+                 "zetenex": zetenex_shape, "qwen2": qwen2_shape}
 # the existing model that a design is set beside: Tudasun beside Koronex, the other design with a recurrent mixer over
 # a float32 state, softmax attention with a sink, layers that read another layer's rows and a per-layer token input
 # Rizovik beside Tudasun: routed feed-forwards, a recurrent mixer over a float32 state, attention over a cache that keeps
 # every row
-BESIDE = {"koronex": "qwen2", "dotivik": "qwen2", "tudasun": "koronex", "rizovik": "tudasun"}
+# Zetenex beside Koronex: a recurrence over a float32 state, softmax attention with a gate, a plain feed-forward (up,
+# activation, down)
+BESIDE = {"koronex": "qwen2", "dotivik": "qwen2", "tudasun": "koronex", "rizovik": "tudasun", "zetenex": "koronex"}
 
 
 def compare_architectures(sizes=("2k", "4k"), design: str = "koronex", beside: str | None = None, **kw) -> dict:
-    """``design`` (Koronex, Dotivik or Tudasun) beside another model (``beside``; default: the Qwen2 dense model, for
-    Tudasun Koronex) at equal width, heads, feed-forward width and count of layer runs."""
+    """``design`` beside another model (``beside``; default: the one BESIDE names) at equal width, heads, feed-forward
+    width and count of layer runs."""
     beside = beside or BESIDE[design]
     out = {"peaks": peaks(), "beside": beside, "sizes": {}}
     for name in sizes:

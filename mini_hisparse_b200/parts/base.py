@@ -173,6 +173,13 @@ class Runtime:
         K.glu_act(gu.tensor, out, activation, nsplit=gu.nsplit, split_stride=gu.split_stride, block=block)
         return out
 
+    def linear_act(self, x, weight, activation: str, ws: Workspace, name: str) -> torch.Tensor:
+        """act(x W^T) in the compute dtype, the activation taken in float32 on the product's float32 output."""
+        z = self.linear(x, weight, ws, name + "_up", out_dtype=torch.float32)
+        out = ws.get(name, (x.shape[0], weight.shape[0]), self.dtype)
+        K.act_rows(z.tensor, out, activation, nsplit=z.nsplit, split_stride=z.split_stride)
+        return out
+
     def linear_swiglu(self, x, weight, block: int, ws: Workspace, name: str) -> torch.Tensor:
         """silu(x Wg^T) * (x Wu^T) in the compute dtype."""
         gu = self.linear(x, weight, ws, name + "_gu")

@@ -83,12 +83,12 @@ class ActivatedMLP(FeedForward):
 
     def forward(self, h, ctx: StepContext) -> Product:
         rt, ws = ctx.rt, ctx.ws
-        z = rt.linear(h, self.up, ws, "ff_up", out_dtype=torch.float32)
-        act = ws.get("ff_act", (h.shape[0], self.inter), rt.dtype)
         if self.polynorm:
+            z = rt.linear(h, self.up, ws, "ff_up", out_dtype=torch.float32)
+            act = ws.get("ff_act", (h.shape[0], self.inter), rt.dtype)
             K.polynorm_rows(z.tensor, self.coef, self.eps, act, nsplit=z.nsplit, split_stride=z.split_stride)
         else:
-            K.act_rows(z.tensor, act, self.activation, nsplit=z.nsplit, split_stride=z.split_stride)
+            act = rt.linear_act(h, self.up, self.activation, ws, "ff_act")
         return rt.linear(act, self.down, ws, "ff_out", out_dtype=torch.float32)       # it joins a float32 sum
 
 
