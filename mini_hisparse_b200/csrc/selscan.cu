@@ -197,7 +197,7 @@ template <int N> __device__ __forceinline__ void copy_async_wait() { asm volatil
 // staged at once.  The step's logits are formed here from the small product's rank columns (dt_weight), the lanes of a
 // channel sharing the dot product: one launch less than a product of its own.
 template <int LPC, int RPL, int CH, int THREADS, typename WT, typename OT>
-__global__ void __launch_bounds__(THREADS, 4)
+__global__ void __launch_bounds__(THREADS, 7)
 selective_step_kernel(const ScanArgs a) {
     constexpr int CPB = THREADS / LPC;                           // channels per CTA
     constexpr int E = (CH * CPB + THREADS - 1) / THREADS;        // elements a thread loads per stage
@@ -248,6 +248,7 @@ selective_step_kernel(const ScanArgs a) {
             const float* lr = low + tt * a.rank;
             float d = 0.f;
             if (a.rank % 8 == 0) {
+#pragma unroll 4
                 for (int i = sub * 8; i < a.rank; i += LPC * 8) {
                     float wv[8];
                     if constexpr (sizeof(WT) == 2) {
@@ -500,10 +501,10 @@ int launch_step(const ScanArgs& a, int S, cudaStream_t stream) {
 
 template <typename WT>
 int pick_step(const ScanArgs& a, int S, cudaStream_t stream) {
-    if (a.N <= 16) return launch_step<4, 4, 16, WT>(a, S, stream);
-    if (a.N <= 32) return launch_step<4, 8, 16, WT>(a, S, stream);
-    if (a.N <= 64) return launch_step<8, 8, 16, WT>(a, S, stream);
-    if (a.N <= 128) return launch_step<16, 8, 8, WT>(a, S, stream);
+    if (a.N <= 16) return launch_step<4, 4, 4, WT>(a, S, stream);
+    if (a.N <= 32) return launch_step<4, 8, 4, WT>(a, S, stream);
+    if (a.N <= 64) return launch_step<8, 8, 4, WT>(a, S, stream);
+    if (a.N <= 128) return launch_step<16, 8, 4, WT>(a, S, stream);
     if (a.N <= 256) return launch_step<32, 8, 4, WT>(a, S, stream);
     return fail("selective_scan: %d states per channel (up to 256)", a.N);
 }
