@@ -1,4 +1,4 @@
-// Recurrences whose gates read the current token only.
+// Linear recurrences, element by element, with coefficients made from the input row alone (so they can be scanned).
 //
 //   mingru_scan   per channel: z = sigmoid(zl + bz), u = xl + bx, c = u >= 0 ? u + 1/2 : sigmoid(u),
 //                 S <- (1 - z) S + z c, out = S silu(gl): zl, xl, gl are columns of one float32 product

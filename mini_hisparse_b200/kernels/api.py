@@ -1247,7 +1247,7 @@ def delta_scan(q, k, v, beta, decay, state, out, tok_seg, seg_slot, positions, *
                                    c_int(1 if writable else 0), _stream()), "delta_scan")
 
 
-# ---- convolutions over time and recurrences whose gates read the current token (csrc/timeconv.cu, selscan.cu) ----
+# ---- convolutions over time and element-by-element recurrences (csrc/timeconv.cu, selscan.cu) ----
 def _seg_args(ctx):
     return _ptr(ctx.seg_offset), _ptr(ctx.seg_slot), _ptr(ctx.positions)
 

@@ -1,4 +1,4 @@
-"""minGRU: a gated recurrence, element by element, whose gate and candidate read the current token only."""
+"""minGRU: one number per channel and request, blended with a candidate; gate and candidate are functions of the input row."""
 from __future__ import annotations
 
 import torch

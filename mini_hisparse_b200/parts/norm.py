@@ -104,8 +104,8 @@ class LayerNorm(Norm):
 
 @register_norm("dyt")
 class DynamicTanh(Norm):
-    """y = tanh(alpha x) * weight + shift with one stored number alpha: a bounded squashing in place of a norm, which
-    takes no mean and no variance.  Computed in float32 from the float32 residual; pending products are added first.
+    """y = tanh(alpha x) * weight + shift with one stored number alpha: a bounded squashing where other blocks
+    have a norm; no statistic of the row is taken.  Computed in float32 from the float32 residual; pending products are added first.
     Since it works element by element, a convolution over time that follows it runs in the same kernel (forward_conv).
     Parameters: width, weight_name (default "weight").  Tensors: the weight, and beside it "alpha" (a scalar) and "b"."""
 

@@ -1,5 +1,5 @@
-"""The selective scan (Mamba): a diagonal recurrence over a float32 state whose step size, input and output vectors are
-read off the current token."""
+"""The selective scan (Mamba): a diagonal linear recurrence over a float32 state whose step size, input vector and output
+vector are made from the input row."""
 from __future__ import annotations
 
 import math
