@@ -2,7 +2,7 @@
 // and values of different widths (any multiples of 8 up to 128; the tiles are padded to the next
 // multiple of 32), a sink per query head in the softmax's denominator, a gate on the output (per element
 // or per head), softmax weights that keep 16 bits in the value product, several score maps per KV head
-// over shared values, capped scores, values that are the head of the key rows (a latent cache), and
+// over shared values, capped scores, scores biased by the distance, values that are the head of the key rows (a latent cache), and
 // float32 outputs.  Work items, tile heights and the merge of
 // key splits are those of attention_mma.cu.
 #include "attention_mma_kernel.cuh"
@@ -49,8 +49,10 @@ int attention_mma_options(const void* q, const void* cache, void* out, float* pa
                                      long long gate_split_stride, int gate_ld, int kparts, float softcap,
                                      int shared_kv, int gate_per_head, int out_f32, int pre_kind, int pre_n,
                                      int value_head, long long out_plane, long long part_plane_rows,
-                                     long long counters_plane, cudaStream_t stream) {
+                                     long long counters_plane, const float* slopes, cudaStream_t stream) {
     if (launch_items <= 0) return 0;
+    if (slopes && (pre_kind || softcap > 0.f)) return fail("attention: distance biases go with uncapped scores inside the window only");
+    if (slopes && !(scale > 0.f)) return fail("attention_mma_ext: distance biases need a positive scale");
     if (pre_kind < 0 || pre_kind > 2 || (pre_kind && pre_n < 1)) return fail("attention: keys beyond the window of kind %d over %d positions", pre_kind, pre_n);
     if ((pre_kind || value_head >= 0) && (kparts != 1 || shared_kv)) return fail("attention: keys beyond the window and another head's values go with plain key and value rows only");
     if (value_head >= nkv || value_head < -2) return fail("attention: values of KV head %d of %d", value_head, nkv);
@@ -66,6 +68,7 @@ int attention_mma_options(const void* q, const void* cache, void* out, float* pa
     a.d = d; a.dv = dv; a.sink = sink; a.gate = gate; a.gate_nsplit = gate_nsplit; a.gate_ld = gate_ld;
     a.gate_split_stride = (size_t)gate_split_stride;
     a.kparts = kparts; a.softcap = softcap; a.shared_kv = shared_kv; a.gate_per_head = gate_per_head; a.out_f32 = out_f32;
+    a.slopes = slopes;
     a.pre_kind = pre_kind; a.pre_n = pre_n; a.vhead = value_head < 0 ? -1 : value_head;
     if (value_head == -2) {          // every KV head's values, a plane of outputs each
         if (nkv > 65535) return fail("attention: too many KV heads for a plane each");
@@ -88,11 +91,12 @@ MHB_EXPORT int mhb_attention_mma_ext(const void* q, const void* cache, void* out
                                      int nkv, int d, int dv, int P, int num_pages, int window, float scale,
                                      const float* sink, const float* gate, int gate_nsplit,
                                      long long gate_split_stride, int gate_ld, int kparts, float softcap,
-                                     int shared_kv, int gate_per_head, int out_f32, cudaStream_t stream) {
+                                     int shared_kv, int gate_per_head, int out_f32, const float* slopes,
+                                     cudaStream_t stream) {
     return attention_mma_options(q, cache, out, part_acc, part_ml, items, num_items, launch_items, rows, positions,
                                  block_table, width, tok_part_row, tok_nsplit, counters, nq, nkv, d, dv, P, num_pages,
                                  window, scale, sink, gate, gate_nsplit, gate_split_stride, gate_ld, kparts, softcap,
-                                 shared_kv, gate_per_head, out_f32, 0, 0, -1, 0, 0, 0, stream);
+                                 shared_kv, gate_per_head, out_f32, 0, 0, -1, 0, 0, 0, slopes, stream);
 }
 
 // The same with keys that stay visible beyond the window (pre_kind 1: the first pre_n positions; 2: the means of
@@ -111,5 +115,6 @@ MHB_EXPORT int mhb_attention_mma_masked(const void* q, const void* cache, void* 
     return attention_mma_options(q, cache, out, part_acc, part_ml, items, num_items, launch_items, rows, positions,
                                  block_table, width, tok_part_row, tok_nsplit, counters, nq, nkv, d, dv, P, num_pages,
                                  window, scale, nullptr, gate, gate_nsplit, gate_split_stride, gate_ld, 1, 0.f, 0, 0,
-                                 out_f32, pre_kind, pre_n, value_head, out_plane, part_plane_rows, counters_plane, stream);
+                                 out_f32, pre_kind, pre_n, value_head, out_plane, part_plane_rows, counters_plane, nullptr,
+                                 stream);
 }

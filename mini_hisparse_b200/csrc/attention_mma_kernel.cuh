@@ -66,6 +66,7 @@ struct AttnArgs {
     // own of the output, of the partial buffers and of the merge counters
     int vplanes;
     size_t out_plane, part_plane_rows, counters_plane;
+    const float* slopes;        // [nq] or null: slope_h * (query position - key position) is taken off the scaled score
 };
 
 __device__ __forceinline__ void store_out(const AttnArgs& a, size_t idx, float v) {
@@ -105,7 +106,8 @@ struct Layout {
 // it lost), which keeps 16 bits of them instead of 8.  Further, with a.kparts > 1 every KV head has that many
 // score maps (gridDim.y = nkv * kparts; query head q belongs to map q % kparts; the maps' keys lie side by side
 // in the key row and share the values), a.softcap caps the scores, a.shared_kv takes the values from the head
-// of the key rows (a latent cache), a.gate_per_head reads one gate per head, a.out_f32 writes float32.
+// of the key rows (a latent cache), a.gate_per_head reads one gate per head, a.out_f32 writes float32, a.slopes biases the scores by
+// the distance.
 template <int D, int DV, int ROWS, bool EXT>
 __global__ void __launch_bounds__(THREADS)
 attention_mma_kernel(const AttnArgs a_in) {
@@ -241,7 +243,15 @@ attention_mma_kernel(const AttnArgs a_in) {
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
     uint32_t qf[Q_IN_REGS ? KSTEPS : 1][4];
     const float scale_log2 = a.scale * 1.4426950408889634f;
+    float slope[2] = {0.f, 0.f};          // in the raw products' units, as the sink below
     if constexpr (EXT) {
+        if (a.slopes) {
+#pragma unroll
+            for (int h = 0; h < 2; ++h) {
+                const int row = wrow + (lane >> 2) + 8 * h;
+                if (row < nrows) slope[h] = a.slopes[head_of(row)] / a.scale;
+            }
+        }
         // the sink is a score that is not scaled: in the units of the raw products it is sink / scale.  It
         // is added a single time per row: in one warp (where four warps share the rows) and one thread of the quad.
         if (a.sink && split <= 0 && (!SPLIT_KEYS || warp == 0)) {
@@ -338,6 +348,7 @@ attention_mma_kernel(const AttnArgs a_in) {
                 const int qp = row_pos[row];
                 bool valid = kp < kv_end && kp <= qp && (a.window <= 0 || kp > qp - a.window);
                 if (EXT && pre) valid = kp < pre_lim[x >> 1];
+                if (EXT && a.slopes) s[j][x] = fmaf(-slope[x >> 1], (float)(qp - kp), s[j][x]);
                 s[j][x] = valid ? s[j][x] : -INFINITY;
                 mx[x >> 1] = fmaxf(mx[x >> 1], s[j][x]);
             }
@@ -584,6 +595,7 @@ inline void fill_args(AttnArgs& a, const void* q, const void* cache, void* out, 
     a.d = a.dv = 0; a.sink = nullptr; a.gate = nullptr; a.gate_nsplit = 1; a.gate_ld = 0; a.gate_split_stride = 0;
     a.kparts = 1; a.softcap = 0.f; a.shared_kv = 0; a.gate_per_head = 0; a.out_f32 = 0;
     a.pre_kind = 0; a.pre_n = 0; a.pool_slots = 0; a.page_extra = 0; a.vhead = -1;
+    a.slopes = nullptr;
     a.vplanes = 0; a.out_plane = a.part_plane_rows = a.counters_plane = 0;
 }
 }  // namespace mhb_amma

@@ -37,6 +37,7 @@
 //                          values of its P positions a page holds [nkv][slots][d] pooled keys and
 //                          [nkv][slots][dv] pooled values, slots = ceil(P / pre_n); block b lies in the page
 //                          of its last position, at slot b - floor(page * P / pre_n))
+//   slopes     one number per query head: slope_h * (query position - key position) is taken off the scaled score
 //   vheads     nkv instead of 1: a query head's weights are applied to the values of EVERY KV head, and the
 //              output row is [nkv][dv] wide (for a mixer that mixes the heads' weights afterwards)
 #include "common.cuh"
@@ -79,6 +80,7 @@ struct AttnArgs {
     int vheads;                // 1, or nkv: values of every KV head
     int vhead;                 // >= 0 (with vheads 1): the values of this KV head, whatever the query head's own
     size_t page_extra;         // elements of a page behind its keys and values
+    const float* slopes;       // [nq] distance biases, or null
 };
 
 __device__ __forceinline__ float gate_of(const AttnArgs& a, int t, int col) {
@@ -135,7 +137,7 @@ attention_simt_kernel(const AttnArgs a) {
     }
     __syncthreads();
 
-    float m[ROWS_PER_WARP], l[ROWS_PER_WARP], acc[ROWS_PER_WARP][DPL];
+    float m[ROWS_PER_WARP], l[ROWS_PER_WARP], acc[ROWS_PER_WARP][DPL], slope[ROWS_PER_WARP];
 #pragma unroll
     for (int rs = 0; rs < ROWS_PER_WARP; ++rs) {
         m[rs] = -INFINITY;
@@ -143,6 +145,7 @@ attention_simt_kernel(const AttnArgs a) {
 #pragma unroll
         for (int i = 0; i < DPL; ++i) acc[rs][i] = 0.f;
         const int r = rs * WARPS + warp;
+        slope[rs] = a.slopes && r < nrows ? a.slopes[(kvh * groups + head0 + r % nheads) * kparts + map] : 0.f;
         if (a.sink && split <= 0 && r < nrows) {      // a single time per token: here or in split 0
             m[rs] = a.sink[(kvh * groups + head0 + r % nheads) * kparts + map];
             l[rs] = 1.f;
@@ -209,6 +212,7 @@ attention_simt_kernel(const AttnArgs a) {
             for (int e = 0; e < d; ++e) s = fmaf(qr[e], kr[e], s);
             s *= a.scale;
             if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
+            if (a.slopes) s = fmaf(-slope[rs], (float)(qp - kp), s);
             bool valid;
             if (phase) valid = kp < end && kp <= qp && (a.window <= 0 || kp > qp - a.window);
             else if (pooled) valid = kp < end && qp - a.window + 1 > 0 && kp < (qp - a.window + 1) / a.pre_n;
@@ -359,6 +363,7 @@ MHB_EXPORT int mhb_attention_simt(const void* q, const void* cache, void* out, i
     a.dv = d; a.sink = nullptr; a.gate = nullptr; a.gate_nsplit = 1; a.gate_ld = 0; a.gate_split_stride = 0;
     a.kparts = 1; a.softcap = 0.f; a.shared_kv = 0; a.gate_per_head = 0; a.out_f32 = 0;
     a.pre_kind = 0; a.pre_n = 0; a.pool_slots = 0; a.vheads = 1; a.page_extra = 0; a.vhead = -1;
+    a.slopes = nullptr;
     MHB_DISPATCH_DTYPE(dtype, CT, return launch_attention<CT>(a, max_items, stream));
     return 0;
 }
@@ -372,8 +377,9 @@ int attention_simt_options(const void* q, const void* cache, void* out, int dtyp
                                       int num_pages, int window, float scale, const float* sink,
                                       const float* gate, int gate_nsplit, long long gate_split_stride, int gate_ld,
                                       int kparts, float softcap, int shared_kv, int gate_per_head, int out_f32,
-                                      int pre_kind, int pre_n, int all_values, cudaStream_t stream) {
+                                      int pre_kind, int pre_n, int all_values, const float* slopes, cudaStream_t stream) {
     if (max_items <= 0) return 0;
+    if (slopes && (pre_kind || softcap > 0.f)) return fail("attention: distance biases go with uncapped scores inside the window only");
     if (pre_kind < 0 || pre_kind > 2 || (pre_kind && pre_n < 1)) return fail("attention: keys beyond the window of kind %d over %d positions", pre_kind, pre_n);
     if ((pre_kind || all_values) && (kparts != 1 || shared_kv)) return fail("attention: keys beyond the window and values of every KV head go with plain key and value rows only");
     if (kparts < 1 || nq % (nkv > 0 ? nkv * kparts : 1)) return fail("attention: %d query heads over %d KV heads with %d score maps each", nq, nkv, kparts);
@@ -396,6 +402,7 @@ int attention_simt_options(const void* q, const void* cache, void* out, int dtyp
     if (a.vhead >= nkv) return fail("attention: values of KV head %d of %d", a.vhead, nkv);
     a.pool_slots = pre_kind == 2 ? (P + pre_n - 1) / pre_n : 0;
     a.page_extra = (size_t)nkv * a.pool_slots * (d + dv);
+    a.slopes = slopes;
     MHB_DISPATCH_DTYPE(dtype, CT, return launch_attention<CT>(a, max_items, stream));
     return 0;
 }
@@ -408,11 +415,11 @@ MHB_EXPORT int mhb_attention_simt_ext(const void* q, const void* cache, void* ou
                                       int num_pages, int window, float scale, const float* sink,
                                       const float* gate, int gate_nsplit, long long gate_split_stride, int gate_ld,
                                       int kparts, float softcap, int shared_kv, int gate_per_head, int out_f32,
-                                      cudaStream_t stream) {
+                                      const float* slopes, cudaStream_t stream) {
     return attention_simt_options(q, cache, out, dtype, part_acc, part_ml, items, num_items, max_items, positions,
                                   block_table, width, tok_part_row, nq, nkv, d, dv, P, num_pages, window, scale, sink,
                                   gate, gate_nsplit, gate_split_stride, gate_ld, kparts, softcap, shared_kv,
-                                  gate_per_head, out_f32, 0, 0, 0, stream);
+                                  gate_per_head, out_f32, 0, 0, 0, slopes, stream);
 }
 
 // The same with keys that stay visible beyond the window (pre_kind, pre_n) and with the values of every KV head
@@ -428,7 +435,7 @@ MHB_EXPORT int mhb_attention_simt_masked(const void* q, const void* cache, void*
     return attention_simt_options(q, cache, out, dtype, part_acc, part_ml, items, num_items, max_items, positions,
                                   block_table, width, tok_part_row, nq, nkv, d, dv, P, num_pages, window, scale, sink,
                                   gate, gate_nsplit, gate_split_stride, gate_ld, 1, 0.f, 0, 0, out_f32, pre_kind,
-                                  pre_n, all_values, stream);
+                                  pre_n, all_values, nullptr, stream);
 }
 
 // every > 0: token t has `every` parts in the rows t * every ... of the partial buffers (tok_part_row and

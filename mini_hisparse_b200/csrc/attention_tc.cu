@@ -69,6 +69,7 @@ struct AttnArgs {
     int shared_kv;
     float softcap;               // s <- softcap * tanh(s / softcap) on the scaled score (0: none)
     int out_f32;                 // `out` is float32 (a sum of the outputs is still to be taken in 32 bits)
+    const float* slopes;         // [nq] or null: slope_h * (query position - key position) is taken off the scaled score
 };
 
 __device__ __forceinline__ float gate_of(const AttnArgs& a, int t, int col) {
@@ -297,7 +298,9 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnArgs a
         const uint32_t lane_addr = tmem + ((uint32_t)(quarter * 32) << 16);
         float m_ref = -INFINITY;      // the maximum the exponentials refer to (at most 2^8 below the true one)
         float l_run = 0.f;
+        float slope = 0.f;            // in the raw products' units
         if constexpr (EXT) {
+            if (a.slopes && live) slope = a.slopes[hq] / a.scale;
             if (a.sink && live && split <= 0) {      // the sink is not scaled: in the raw products' units it is sink / scale
                 m_ref = a.sink[hq] / a.scale;
                 l_run = 1.f;
@@ -325,6 +328,14 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnArgs a
                 }
             }
             const int t0 = tile_begin + j * KT;
+            if constexpr (EXT) {
+                if (a.slopes) {               // distances are exact in float32
+                    const float ahead = live ? (float)(t0 - qp) : 0.f;
+#pragma unroll
+                    for (int x = 0; x < KT; ++x)
+                        sr[x] = __float_as_uint(fmaf(slope, ahead + (float)x, __uint_as_float(sr[x])));
+                }
+            }
             // most tiles lie wholly inside this row's range of keys: no mask then
             const int lo = max(kv_begin, a.window > 0 ? qp - a.window + 1 : 0), hi = min(kv_end - 1, qp);
             if (!(t0 >= lo && t0 + KT - 1 <= hi)) {
@@ -513,7 +524,7 @@ MHB_EXPORT int mhb_attention_tc(const void* q, const void* cache, void* out, con
     a.status = status; a.num_items = num_items; a.width = width; a.nq = nq;
     a.nkv = nkv; a.P = P; a.num_pages = num_pages; a.window = window; a.scale = scale;
     a.sink = nullptr; a.gate = nullptr; a.gate_nsplit = 1; a.gate_ld = 0; a.gate_split_stride = 0;
-    a.gate_per_head = 0; a.shared_kv = 0; a.softcap = 0.f; a.out_f32 = 0;
+    a.gate_per_head = 0; a.shared_kv = 0; a.softcap = 0.f; a.out_f32 = 0; a.slopes = nullptr;
     return d == 128 ? launch<128, false>(map, a, num_items, stream) : launch<64, false>(map, a, num_items, stream);
 }
 
@@ -526,13 +537,14 @@ MHB_EXPORT int mhb_attention_tc_ext(const void* q, const void* cache, void* out,
                                     const int* tok_part_row, float* part_acc, float* part_ml, int nq, int nkv, int d,
                                     int P, int num_pages, int window, float scale, const float* sink,
                                     const float* gate, int gate_nsplit, long long gate_split_stride, int gate_ld,
-                                    int gate_per_head, int shared_kv, float softcap, int out_f32, int* status,
-                                    cudaStream_t stream) {
+                                    int gate_per_head, int shared_kv, float softcap, int out_f32,
+                                    const float* slopes, int* status, cudaStream_t stream) {
     if (num_items <= 0) return 0;
     if (nkv <= 0 || nq % nkv) return fail("attention: %d query heads over %d KV heads", nq, nkv);
     if (!mhb_attention_tc_supports(d, P))
         return fail("attention_tc: head_dim %d with pages of %d keys is not built (head_dim 64 or 128, page size dividing 64)", d, P);
-    if (sink && !(scale > 0.f)) return fail("attention_tc: a sink needs a positive scale");
+    if ((sink || slopes) && !(scale > 0.f)) return fail("attention_tc: a sink and distance biases need a positive scale");
+    if (slopes && softcap > 0.f) return fail("attention_tc: distance biases go with uncapped scores only");
     if (shared_kv && nkv != 1) return fail("attention_tc: rows that are key and value at once have one KV head");
     const long long total_rows = shared_kv ? (long long)num_pages * P : (long long)num_pages * 2 * nkv * P;
     if (total_rows > 0x7fffffffLL) return fail("attention_tc: the pool has too many rows for one tensor map");
@@ -547,5 +559,6 @@ MHB_EXPORT int mhb_attention_tc_ext(const void* q, const void* cache, void* out,
     a.sink = sink; a.gate = gate; a.gate_nsplit = gate_nsplit; a.gate_ld = gate_ld;
     a.gate_split_stride = (size_t)gate_split_stride;
     a.gate_per_head = gate_per_head; a.shared_kv = shared_kv; a.softcap = softcap; a.out_f32 = out_f32;
+    a.slopes = slopes;
     return d == 128 ? launch<128, true>(map, a, num_items, stream) : launch<64, true>(map, a, num_items, stream);
 }

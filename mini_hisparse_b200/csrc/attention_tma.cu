@@ -54,6 +54,7 @@ struct AttnArgs {
     int shared_kv;              // a latent cache: the pool is [pages][P][d] rows (one KV head), a row is key AND value
     float softcap;              // s <- softcap * tanh(s / softcap) on the scaled score (0: none)
     int out_f32;                // `out` is float32 (a sum of the outputs is still to be taken in 32 bits)
+    const float* slopes;        // [nq] or null: slope_h * (query position - key position) is taken off the scaled score
 };
 
 __device__ __forceinline__ void store_out(const AttnArgs& a, size_t idx, float v) {
@@ -207,7 +208,15 @@ attention_tma_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnArgs 
 #pragma unroll
     for (int i = 0; i < DTILES; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
+    float slope[2] = {0.f, 0.f};          // in the raw products' units
     if constexpr (EXT) {
+        if (a.slopes) {
+#pragma unroll
+            for (int h = 0; h < 2; ++h) {
+                const int row = wrow + (lane >> 2) + 8 * h;
+                if (row < nrows) slope[h] = a.slopes[kvh * groups + head0 + row % nheads] / a.scale;
+            }
+        }
         if (a.sink && split <= 0 && (!SPLIT_KEYS || warp == 0)) {
 #pragma unroll
             for (int h = 0; h < 2; ++h) {
@@ -269,6 +278,7 @@ attention_tma_kernel(const __grid_constant__ CUtensorMap kv_map, const AttnArgs 
                 const int kp = t0 + key0 + j * 8 + (lane & 3) * 2 + (x & 1);
                 const int qp = row_pos[row];
                 const bool valid = kp >= kv_begin && kp < kv_end && kp <= qp && (a.window <= 0 || kp > qp - a.window);
+                if (EXT && a.slopes) s[j][x] = fmaf(-slope[x >> 1], (float)(qp - kp), s[j][x]);
                 s[j][x] = valid ? s[j][x] : -INFINITY;
                 mx[x >> 1] = fmaxf(mx[x >> 1], s[j][x]);
             }
@@ -550,7 +560,7 @@ MHB_EXPORT int mhb_attention_tma(const void* q, const void* cache, void* out, fl
     a.width = width; a.nq = nq; a.nkv = nkv; a.P = P; a.num_pages = num_pages; a.window = window;
     a.scale = scale;
     a.fresh = fresh;
-    a.gate_per_head = 0; a.shared_kv = 0; a.softcap = 0.f; a.out_f32 = 0;
+    a.gate_per_head = 0; a.shared_kv = 0; a.softcap = 0.f; a.out_f32 = 0; a.slopes = nullptr;
     a.sink = nullptr; a.gate = nullptr; a.gate_nsplit = 1; a.gate_ld = 0; a.gate_split_stride = 0;
     if (rows == 16) return d == 128 ? launch<128, 16, false>(map, a, launch_items, stream) : launch<64, 16, false>(map, a, launch_items, stream);
     return fail("attention_tma: tile height %d", rows);
@@ -564,12 +574,14 @@ MHB_EXPORT int mhb_attention_tma_ext(const void* q, const void* cache, void* out
                                      int d, int P, int num_pages, int window, int fresh, float scale,
                                      const float* sink, const float* gate, int gate_nsplit,
                                      long long gate_split_stride, int gate_ld, int gate_per_head, int shared_kv,
-                                     float softcap, int out_f32, int* status, cudaStream_t stream) {
+                                     float softcap, int out_f32, const float* slopes, int* status,
+                                     cudaStream_t stream) {
     if (launch_items <= 0) return 0;
     if (nkv <= 0 || nq % nkv) return fail("attention: %d query heads over %d KV heads", nq, nkv);
     if (!mhb_attention_tma_supports(d, P))
         return fail("attention_tma: head_dim %d with pages of %d keys is not built (head_dim 64 or 128, page size dividing 64)", d, P);
-    if (sink && !(scale > 0.f)) return fail("attention_tma: a sink needs a positive scale");
+    if ((sink || slopes) && !(scale > 0.f)) return fail("attention_tma: a sink and distance biases need a positive scale");
+    if (slopes && softcap > 0.f) return fail("attention_tma: distance biases go with uncapped scores only");
     if (shared_kv && nkv != 1) return fail("attention_tma: rows that are key and value at once have one KV head");
     const long long total_rows = shared_kv ? (long long)num_pages * P : (long long)num_pages * 2 * nkv * P;
     if (total_rows > 0x7fffffffLL) return fail("attention_tma: the pool has too many rows for one tensor map");
@@ -586,6 +598,7 @@ MHB_EXPORT int mhb_attention_tma_ext(const void* q, const void* cache, void* out
     a.sink = sink; a.gate = gate; a.gate_nsplit = gate_nsplit; a.gate_ld = gate_ld;
     a.gate_split_stride = (size_t)gate_split_stride;
     a.gate_per_head = gate_per_head; a.shared_kv = shared_kv; a.softcap = softcap; a.out_f32 = out_f32;
+    a.slopes = slopes;
     if (rows == 16) return d == 128 ? launch<128, 16, true>(map, a, launch_items, stream) : launch<64, 16, true>(map, a, launch_items, stream);
     return fail("attention_tma: tile height %d", rows);
 }

@@ -72,6 +72,39 @@ MHB_EXPORT int mhb_embed_scaled(const void* table, int table_dtype, const int* t
     return launch_embed(table, table_dtype, tokens, out, T, H, V, status, scale, copy, stream);
 }
 
+// out[t, :] = rms(table[tokens[t], :]) * weight: an embedding whose rows are normalised as they enter the stream
+template <typename WT>
+__global__ void embed_norm_kernel(const WT* __restrict__ table, const int* __restrict__ tokens,
+                                  const float* __restrict__ weight, float eps, float* __restrict__ out, int H, int V,
+                                  int* __restrict__ status) {
+    __shared__ float scratch[33];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x;
+    const int tok = tokens[t];
+    float* o = out + (size_t)t * H;
+    if (tok < 0 || tok >= V) {
+        for (int i = threadIdx.x; i < H; i += blockDim.x) o[i] = 0.f;
+        if (threadIdx.x == 0 && status) atomicOr(status, 1);
+        return;
+    }
+    const WT* row = table + (size_t)tok * H;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < H; i += blockDim.x) { const float v = to_float(row[i]); ss += v * v; }
+    const float rstd = 1.f / sqrtf(block_sum(ss, scratch) / (float)H + eps);
+    for (int i = threadIdx.x; i < H; i += blockDim.x) o[i] = to_float(row[i]) * rstd * weight[i];
+}
+
+MHB_EXPORT int mhb_embed_norm(const void* table, int table_dtype, const int* tokens, const float* weight, float eps,
+                              float* out, int T, int H, int V, int* status, cudaStream_t stream) {
+    if (T <= 0) return 0;
+    const int threads = H >= 1024 ? 256 : 128;
+    MHB_DISPATCH_DTYPE(table_dtype, WT,
+        launch_kernel(embed_norm_kernel<WT>, dim3(T), dim3(threads), 0, stream, (const WT*)table, tokens, weight, eps, out,
+                      H, V, status));
+    return check_launch("embed_norm");
+}
+
 // ---- (add +) RMSNorm -----------------------------------------------------------------------
 // For output row r (source row s = rows ? rows[r] : r):
 //   v = x[s] (+ delta[s]);  if delta and !rows: x[s] = v  (residual updated in place)

@@ -156,10 +156,16 @@ template <> __device__ __forceinline__ void store_out<__nv_bfloat16>(__nv_bfloat
 
 // EPI 1 and 3 are the gated epilogues: act(gate) * up with act = silu (1) or the tanh form of gelu (3).
 __host__ __device__ constexpr bool is_glu(int epi) { return epi == 1 || epi == 3; }
-// EPI 4 applies the tanh form of gelu to every element (no gate).
+// EPI 4, 5 and 6 apply an activation to every element (no gate): the tanh form of gelu, the exact gelu, the square of relu.
 __device__ __forceinline__ float gelu_tanh(float g) {
     const float c = 0.7978845608028654f;      // sqrt(2 / pi)
     return 0.5f * g * (1.f + tanhf(c * (g + 0.044715f * g * g * g)));
+}
+template <int EPI>
+__device__ __forceinline__ float plain_act(float z) {
+    if constexpr (EPI == 4) return gelu_tanh(z);
+    else if constexpr (EPI == 5) return 0.5f * z * (1.f + erff(z * 0.7071067811865476f));
+    else { const float a = fmaxf(z, 0.f); return a * a; }
 }
 template <int EPI>
 __device__ __forceinline__ float glu_mul(float g, float u) {
@@ -437,9 +443,9 @@ template <typename OT, int EPI>
 __device__ __forceinline__ void emit_unit(OT* __restrict__ C, long long ldc, int Ra, int Rb, int ra, int rb0, int c0,
                                           uint32_t (&r)[16], const uint32_t (&r2)[16]) {
     if (ra >= Ra) return;
-    if constexpr (EPI == 4) {
+    if constexpr (EPI >= 4 && EPI <= 6) {
 #pragma unroll
-        for (int x = 0; x < 16; ++x) r[x] = __float_as_uint(gelu_tanh(__uint_as_float(r[x])));
+        for (int x = 0; x < 16; ++x) r[x] = __float_as_uint(plain_act<EPI>(__uint_as_float(r[x])));
     }
     if constexpr (is_glu(EPI)) {
         OT* row = C + (size_t)ra * ldc + (rb0 + c0) / 2;
@@ -1522,13 +1528,15 @@ MHB_EXPORT int mhb_gemm_tc_glu(const void* X, const void* W, void* C, int c_dtyp
     return fail("gemm_tc_glu: unknown activation %d", act);
 }
 
-// C[M, N] = act(X W^T), bfloat16 out, the activation (1 = the tanh form of gelu) taken in float32 on the accumulators in
+// C[M, N] = act(X W^T), bfloat16 out, the activation (1 = the tanh form of gelu, 2 = the exact gelu, 3 = the square of relu) taken in float32 on the accumulators in
 // the persistent product's epilogue (more than 64 tokens).
 MHB_EXPORT int mhb_gemm_tc_act(const void* X, const void* W, void* C, int M, int N, int K, long long lda, long long ldw,
                                long long ldc, float* partials, int* flags, int* status, int act, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
-    if (act != 1) return fail("gemm_tc_act: unknown activation %d", act);
+    if (act < 1 || act > 3) return fail("gemm_tc_act: unknown activation %d", act);
     if (K <= 0 || K % 8 || lda % 8 || ldw % 8) return fail("gemm_tc: K, lda and ldw must be multiples of 8 (K %d, lda %lld, ldw %lld)", K, lda, ldw);
     if (((uintptr_t)X & 15) || ((uintptr_t)W & 15)) return fail("gemm_tc: operands must be 16-byte aligned");
-    return launch_persistent<__nv_bfloat16, 4>(X, W, C, M, N, K, lda, ldw, ldc, partials, flags, status, stream);
+    if (act == 1) return launch_persistent<__nv_bfloat16, 4>(X, W, C, M, N, K, lda, ldw, ldc, partials, flags, status, stream);
+    if (act == 2) return launch_persistent<__nv_bfloat16, 5>(X, W, C, M, N, K, lda, ldw, ldc, partials, flags, status, stream);
+    return launch_persistent<__nv_bfloat16, 6>(X, W, C, M, N, K, lda, ldw, ldc, partials, flags, status, stream);
 }

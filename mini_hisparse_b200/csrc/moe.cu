@@ -1,15 +1,16 @@
 // A routed feed-forward (mixture of experts) without a word from the host between its kernels:
 //
-//   moe_route     per token: softmax over the router's outputs, choice scores (softmax + correction), the best
-//                 `keep` of `groups` equal groups of neighbours, the `top` best choice scores inside them, and
-//                 the chosen outputs' softmax values divided by their sum (+ 1e-20)
+//   moe_route     per token: scores (a softmax over the router's outputs, or a sigmoid of each), choice scores (score +
+//                 correction), the best `keep` of `groups` equal groups of neighbours (by their largest choice score, or
+//                 by the sum of their two largest), the `top` best choice scores inside them, and as weights the chosen
+//                 outputs' scores divided by their sum (+ 1e-20), or times a factor
 //   moe_plan      the chosen (token, expert) pairs grouped by expert: a row per pair, tiles of TILE_ROWS rows of
 //                 one expert each (outputs at or beyond `experts` are identity experts and get no row)
-//   moe_linear    out[r] = W[expert of r] x[source of r], tile by tile; `glu`: W holds [gate ; up] and the result is
-//                 silu(gate x) * (up x).  bfloat16 on mma.sync m16n8k16, float32 (and odd widths) on FFMA tiles;
+//   moe_linear    out[r] = W[expert of r] x[source of r], tile by tile; ACT 1: W holds [gate ; up] and the result is
+//                 silu(gate x) * (up x); ACT 2: the result is the square of relu(W x).  bfloat16 on mma.sync m16n8k16, float32 (and odd widths) on FFMA tiles;
 //                 float32 accumulation in both
 //   moe_combine   out[t] = sum_k weight[t, k] * (row of pair (t, k), or the input itself for an identity expert)
-//                          + sigmoid(shared gate logit[t]) * shared expert's output[t]
+//                          + sigmoid(shared gate logit[t]) * shared expert's output[t]   (no gate: 1)
 //
 // Which row a pair gets inside its expert depends on the order of atomic additions; every row is computed by
 // itself and a token's pairs are summed in the order of their choice, so the result does not.
@@ -35,7 +36,7 @@ __device__ __forceinline__ float load_parts(const float* p, size_t idx, int nspl
 __global__ void __launch_bounds__(128)
 route_kernel(const float* __restrict__ logits, int nsplit, size_t stride, int ld, const float* __restrict__ correction,
              int* __restrict__ chosen, float* __restrict__ weights, int T, int n, int top, int groups, int keep,
-             const float* __restrict__ bias) {
+             const float* __restrict__ bias, int sigmoid, int group_two, int normalise, float factor) {
     extern __shared__ float sm[];
     pdl_launch_dependents();
     pdl_wait();
@@ -54,11 +55,11 @@ route_kernel(const float* __restrict__ logits, int nsplit, size_t stride, int ld
     mx = warp_max(mx);
     float sum = 0.f;
     for (int i = lane; i < n; i += 32) {
-        const float e = expf(s[i] - mx);
+        const float e = sigmoid ? 1.f / (1.f + expf(-s[i])) : expf(s[i] - mx);
         s[i] = e;
         sum += e;
     }
-    sum = warp_sum(sum);
+    sum = sigmoid ? 1.f : warp_sum(sum);
     for (int i = lane; i < n; i += 32) {
         s[i] = s[i] / sum;
         c[i] = s[i] + (correction ? correction[i] : 0.f);
@@ -67,9 +68,13 @@ route_kernel(const float* __restrict__ logits, int nsplit, size_t stride, int ld
     if (groups > 1 && keep < groups) {
         const int per = n / groups;
         for (int g = lane; g < groups; g += 32) {
-            float best = -INFINITY;
-            for (int i = 0; i < per; ++i) best = fmaxf(best, c[g * per + i]);
-            gs[g] = best;
+            float best = -INFINITY, second = -INFINITY;
+            for (int i = 0; i < per; ++i) {
+                const float v = c[g * per + i];
+                second = fmaxf(second, fminf(best, v));
+                best = fmaxf(best, v);
+            }
+            gs[g] = group_two && per > 1 ? best + second : best;
         }
         __syncwarp();
         // the `keep` best groups, ties to the lower index; a taken group's score becomes NaN-free +inf mark
@@ -122,7 +127,7 @@ route_kernel(const float* __restrict__ logits, int nsplit, size_t stride, int ld
         }
     }
     __syncwarp();
-    const float inv = 1.f / (total + 1e-20f);
+    const float inv = normalise ? factor / (total + 1e-20f) : factor;
     for (int k = lane; k < top; k += 32) weights[(size_t)t * top + k] *= inv;
 }
 
@@ -175,14 +180,16 @@ plan_kernel(const int* __restrict__ chosen, int pairs, int top, int experts, int
 }
 
 __device__ __forceinline__ float siluf_(float z) { return z / (1.f + expf(-z)); }
+__device__ __forceinline__ float relu2f_(float z) { const float a = fmaxf(z, 0.f); return a * a; }
 
 // ---- grouped product, CUDA cores ---------------------------------------------------------------------------
 // tile: 32 rows x 64 outputs, K in blocks of 32; 128 threads, 4 x 4 outputs each.  glu: outputs n and F + n of W.
 constexpr int GL_T = 32, GL_N = 64, GL_K = 32;
-template <typename XT, typename OT, bool GLU>
+template <typename XT, typename OT, int ACT>
 __global__ void __launch_bounds__(128)
 linear_kernel(const XT* __restrict__ x, size_t x_ld, const int* __restrict__ plan, int max_tiles, int pairs, int gather,
               const XT* __restrict__ w, OT* __restrict__ out, int N, int K) {
+    constexpr bool GLU = ACT == 1;
     __shared__ float xs[GL_T][GL_K + 1];
     __shared__ float ws[GLU ? 2 : 1][GL_N][GL_K + 1];
     __shared__ int src[GL_T];
@@ -246,7 +253,7 @@ linear_kernel(const XT* __restrict__ x, size_t x_ld, const int* __restrict__ pla
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tx + 16 * j;
             if (n >= N) continue;
-            const float v = GLU ? siluf_(acc[i][j]) * acc2[GLU ? i : 0][j] : acc[i][j];
+            const float v = GLU ? siluf_(acc[i][j]) * acc2[GLU ? i : 0][j] : ACT == 2 ? relu2f_(acc[i][j]) : acc[i][j];
             out[(size_t)r * N + n] = from_float<OT>(v);
         }
     }
@@ -259,10 +266,11 @@ linear_kernel(const XT* __restrict__ x, size_t x_ld, const int* __restrict__ pla
 // tensor cores and by how many CTAs an SM holds: two stages.
 constexpr int GM_N = 64, GM_K = 64, GM_LD = GM_K + 8, GM_FEW_ROWS = 512;
 constexpr size_t gm_smem(bool glu, int stages) { return (size_t)stages * (TILE_ROWS + (glu ? 2 : 1) * GM_N) * GM_LD * 2; }
-template <typename OT, bool GLU, int GM_STAGES>
+template <typename OT, int ACT, int GM_STAGES>
 __global__ void __launch_bounds__(128)
 linear_mma_kernel(const __nv_bfloat16* __restrict__ x, size_t x_ld, const int* __restrict__ plan, int max_tiles,
                   int pairs, int gather, const __nv_bfloat16* __restrict__ w, OT* __restrict__ out, int N, int K) {
+    constexpr bool GLU = ACT == 1;
     extern __shared__ __align__(16) unsigned char gm_stages[];       // [GM_STAGES] x {x tile, w tile}
     __shared__ int src[TILE_ROWS];
     constexpr uint32_t XS_BYTES = TILE_ROWS * GM_LD * 2, STAGE_BYTES = XS_BYTES + (GLU ? 2 : 1) * GM_N * GM_LD * 2;
@@ -350,7 +358,7 @@ linear_mma_kernel(const __nv_bfloat16* __restrict__ x, size_t x_ld, const int* _
             for (int u = 0; u < 2; ++u) {
                 if (n + u >= N) continue;
                 const float a = acc[j][2 * half + u];
-                o[n + u] = from_float<OT>(GLU ? siluf_(a) * acc2[GLU ? j : 0][2 * half + u] : a);
+                o[n + u] = from_float<OT>(GLU ? siluf_(a) * acc2[GLU ? j : 0][2 * half + u] : ACT == 2 ? relu2f_(a) : a);
             }
         }
     }
@@ -368,7 +376,7 @@ combine_kernel(const float* __restrict__ y, const int* __restrict__ plan, int ma
     const size_t t = blockIdx.x;
     const int* pair_row = plan + 1 + 3 * max_tiles + pairs;
     float gate = 0.f;
-    if (shared) gate = 1.f / (1.f + expf(-load_parts(sg, t * g_ld, gn, gs)));
+    if (shared) gate = sg ? 1.f / (1.f + expf(-load_parts(sg, t * g_ld, gn, gs))) : 1.f;
     for (int j = threadIdx.x; j < W; j += blockDim.x) {
         float acc = 0.f;
         for (int k = 0; k < top; ++k) {
@@ -386,11 +394,13 @@ combine_kernel(const float* __restrict__ y, const int* __restrict__ plan, int ma
 
 MHB_EXPORT int mhb_moe_tile_rows() { return TILE_ROWS; }
 
-// bias (or null): added to the logits before the softmax; correction may be null too (no correction).  With both
-// null groups the choice is by the logits themselves and the weights are the softmax over the chosen logits.
-MHB_EXPORT int mhb_moe_route_biased(const float* logits, int nsplit, long long stride, int ld, const float* bias,
+// bias (or null): added to the logits before the scores; correction may be null too (no correction).  sigmoid 0: a softmax
+// over the outputs, 1: each output's sigmoid.  group_two: a group's score is the sum of its two largest choice scores
+// instead of the largest.  normalise: the weights are divided by their sum; factor multiplies them.
+MHB_EXPORT int mhb_moe_route_opts(const float* logits, int nsplit, long long stride, int ld, const float* bias,
                                     const float* correction, int* chosen, float* weights, int T, int n, int top,
-                                    int groups, int keep, cudaStream_t stream) {
+                                    int groups, int keep, int sigmoid, int group_two, int normalise, float factor,
+                                    cudaStream_t stream) {
     if (T <= 0) return 0;
     if (top < 1 || top > n) return fail("moe_route: %d picks among %d outputs", top, n);
     if (groups < 1 || n % groups || keep < 1 || keep > groups)
@@ -400,9 +410,19 @@ MHB_EXPORT int mhb_moe_route_biased(const float* logits, int nsplit, long long s
     const size_t smem = sizeof(float) * warps * (2 * (size_t)n + groups);
     if (smem > 48 * 1024) return fail("moe_route: %d router outputs are more than the kernel holds", n);
     cudaError_t e = launch_kernel(route_kernel, dim3((T + warps - 1) / warps), dim3(32 * warps), smem, stream, logits,
-                                  nsplit, (size_t)stride, ld, correction, chosen, weights, T, n, top, groups, keep, bias);
+                                  nsplit, (size_t)stride, ld, correction, chosen, weights, T, n, top, groups, keep, bias,
+                                  sigmoid, group_two, normalise, factor);
     if (e != cudaSuccess) return fail("moe_route: %s", cudaGetErrorString(e));
     return check_launch("moe_route");
+}
+
+// With a softmax, the largest choice score as a group's, and weights divided by their sum; without a correction and groups
+// the choice is by the logits themselves and the weights are the softmax over the chosen logits.
+MHB_EXPORT int mhb_moe_route_biased(const float* logits, int nsplit, long long stride, int ld, const float* bias,
+                                    const float* correction, int* chosen, float* weights, int T, int n, int top,
+                                    int groups, int keep, cudaStream_t stream) {
+    return mhb_moe_route_opts(logits, nsplit, stride, ld, bias, correction, chosen, weights, T, n, top, groups, keep, 0, 0,
+                              1, 1.f, stream);
 }
 
 MHB_EXPORT int mhb_moe_route(const float* logits, int nsplit, long long stride, int ld, const float* correction,
@@ -424,9 +444,10 @@ MHB_EXPORT int mhb_moe_plan(const int* chosen, int pairs, int top, int experts, 
 }
 
 MHB_EXPORT int mhb_moe_linear(const void* x, int x_dtype, long long x_ld, const int* plan, int max_tiles, int pairs,
-                              int gather, const void* w, void* out, int out_dtype, int N, int K, int glu,
+                              int gather, const void* w, void* out, int out_dtype, int N, int K, int act,
                               cudaStream_t stream) {
     if (pairs <= 0 || max_tiles <= 0) return 0;
+    if (act < 0 || act > 2) return fail("moe_linear: unknown activation %d", act);
     const bool mma = x_dtype == MHB_BF16 && K % 8 == 0 && x_ld % 8 == 0 && ((uintptr_t)x & 15) == 0 && ((uintptr_t)w & 15) == 0;
     cudaError_t e;
     if (mma) {
@@ -434,47 +455,45 @@ MHB_EXPORT int mhb_moe_linear(const void* x, int x_dtype, long long x_ld, const 
         const __nv_bfloat16* xb = (const __nv_bfloat16*)x;
         const __nv_bfloat16* wb = (const __nv_bfloat16*)w;
         const bool few = pairs <= GM_FEW_ROWS;
-        if (glu && out_dtype != MHB_BF16) return fail("moe_linear: the gated product writes the compute dtype");
-#define MHB_MOE_MMA(OT, GLU, ST)                                                                                      \
+        if (act && out_dtype != MHB_BF16) return fail("moe_linear: a product with an activation writes the compute dtype");
+#define MHB_MOE_MMA(OT, ACT, ST)                                                                                      \
     do {                                                                                                              \
         static bool raised = false;                                                                                   \
         if (!raised) {                                                                                                \
-            if (cudaFuncSetAttribute(linear_mma_kernel<OT, GLU, ST>, cudaFuncAttributeMaxDynamicSharedMemorySize,     \
-                                     (int)gm_smem(GLU, ST)) != cudaSuccess)                                           \
+            if (cudaFuncSetAttribute(linear_mma_kernel<OT, ACT, ST>, cudaFuncAttributeMaxDynamicSharedMemorySize,     \
+                                     (int)gm_smem(ACT == 1, ST)) != cudaSuccess)                                           \
                 return fail("moe_linear: cannot raise the shared-memory limit");                                      \
             raised = true;                                                                                            \
         }                                                                                                             \
-        e = launch_kernel(linear_mma_kernel<OT, GLU, ST>, grid, dim3(128), gm_smem(GLU, ST), stream, xb, (size_t)x_ld, \
+        e = launch_kernel(linear_mma_kernel<OT, ACT, ST>, grid, dim3(128), gm_smem(ACT == 1, ST), stream, xb, (size_t)x_ld, \
                           plan, max_tiles, pairs, gather, wb, (OT*)out, N, K);                                        \
     } while (0)
-        if (glu) {
-            if (few) MHB_MOE_MMA(__nv_bfloat16, true, 4); else MHB_MOE_MMA(__nv_bfloat16, true, 2);
+        if (act == 1) {
+            if (few) MHB_MOE_MMA(__nv_bfloat16, 1, 4); else MHB_MOE_MMA(__nv_bfloat16, 1, 2);
+        } else if (act == 2) {
+            if (few) MHB_MOE_MMA(__nv_bfloat16, 2, 4); else MHB_MOE_MMA(__nv_bfloat16, 2, 2);
         } else if (out_dtype == MHB_F32) {
-            if (few) MHB_MOE_MMA(float, false, 4); else MHB_MOE_MMA(float, false, 2);
+            if (few) MHB_MOE_MMA(float, 0, 4); else MHB_MOE_MMA(float, 0, 2);
         } else {
-            if (few) MHB_MOE_MMA(__nv_bfloat16, false, 4); else MHB_MOE_MMA(__nv_bfloat16, false, 2);
+            if (few) MHB_MOE_MMA(__nv_bfloat16, 0, 4); else MHB_MOE_MMA(__nv_bfloat16, 0, 2);
         }
 #undef MHB_MOE_MMA
     } else {
         dim3 grid(max_tiles * (TILE_ROWS / GL_T), (N + GL_N - 1) / GL_N);
+#define MHB_MOE_SIMT(XT, OT, ACT)                                                                                    \
+    launch_kernel(linear_kernel<XT, OT, ACT>, grid, dim3(128), 0, stream, (const XT*)x, (size_t)x_ld, plan, max_tiles, \
+                  pairs, gather, (const XT*)w, (OT*)out, N, K)
         if (x_dtype == MHB_F32) {
             if (out_dtype != MHB_F32) return fail("moe_linear: a float32 product writes float32");
-            e = glu ? launch_kernel(linear_kernel<float, float, true>, grid, dim3(128), 0, stream, (const float*)x,
-                                    (size_t)x_ld, plan, max_tiles, pairs, gather, (const float*)w, (float*)out, N, K)
-                    : launch_kernel(linear_kernel<float, float, false>, grid, dim3(128), 0, stream, (const float*)x,
-                                    (size_t)x_ld, plan, max_tiles, pairs, gather, (const float*)w, (float*)out, N, K);
+            e = act == 1 ? MHB_MOE_SIMT(float, float, 1) : act == 2 ? MHB_MOE_SIMT(float, float, 2) : MHB_MOE_SIMT(float, float, 0);
         } else {
-            const __nv_bfloat16* xb = (const __nv_bfloat16*)x;
-            const __nv_bfloat16* wb = (const __nv_bfloat16*)w;
-            if (glu && out_dtype == MHB_BF16)
-                e = launch_kernel(linear_kernel<__nv_bfloat16, __nv_bfloat16, true>, grid, dim3(128), 0, stream, xb,
-                                  (size_t)x_ld, plan, max_tiles, pairs, gather, wb, (__nv_bfloat16*)out, N, K);
-            else if (!glu && out_dtype == MHB_F32)
-                e = launch_kernel(linear_kernel<__nv_bfloat16, float, false>, grid, dim3(128), 0, stream, xb, (size_t)x_ld,
-                                  plan, max_tiles, pairs, gather, wb, (float*)out, N, K);
+            if (act == 1 && out_dtype == MHB_BF16) e = MHB_MOE_SIMT(__nv_bfloat16, __nv_bfloat16, 1);
+            else if (act == 2 && out_dtype == MHB_BF16) e = MHB_MOE_SIMT(__nv_bfloat16, __nv_bfloat16, 2);
+            else if (!act && out_dtype == MHB_F32) e = MHB_MOE_SIMT(__nv_bfloat16, float, 0);
             else
-                return fail("moe_linear: the gated product writes the compute dtype, the plain one float32");
+                return fail("moe_linear: a product with an activation writes the compute dtype, the plain one float32");
         }
+#undef MHB_MOE_SIMT
     }
     if (e != cudaSuccess) return fail("moe_linear: %s", cudaGetErrorString(e));
     return check_launch("moe_linear");

@@ -34,6 +34,7 @@ __device__ __forceinline__ float load_parts_t(const T* p, size_t idx, int nsplit
 }
 
 __device__ __forceinline__ float sigmoidf(float z) { return 1.f / (1.f + expf(-z)); }
+__device__ __forceinline__ float geluf(float z) { return 0.5f * z * (1.f + erff(z * 0.7071067811865476f)); }
 __device__ __forceinline__ float gelu_tanhf(float z) {
     const float c = 0.7978845608028654f;      // sqrt(2 / pi)
     return 0.5f * z * (1.f + tanhf(c * (z + 0.044715f * z * z * z)));
@@ -133,7 +134,15 @@ __global__ void norm_mix_vec_kernel(float* __restrict__ x, const DT* __restrict_
 }
 
 // ---- activations of a product ----------------------------------------------------------------------
-enum { ACT_RELU2 = 0, ACT_SILU = 1, ACT_GELU_TANH = 2, ACT_COPY = 3 };
+enum { ACT_RELU2 = 0, ACT_SILU = 1, ACT_GELU_TANH = 2, ACT_COPY = 3, ACT_GELU = 4 };
+
+__device__ __forceinline__ float act_of(float v, int act) {
+    if (act == ACT_RELU2) { const float a = fmaxf(v, 0.f); return a * a; }
+    if (act == ACT_SILU) return v * sigmoidf(v);
+    if (act == ACT_GELU_TANH) return gelu_tanhf(v);
+    if (act == ACT_GELU) return geluf(v);
+    return v;
+}
 
 template <typename IT, typename OT>
 __global__ void act_rows_kernel(const IT* __restrict__ z, int nsplit, size_t split_stride, OT* __restrict__ out,
@@ -143,19 +152,7 @@ __global__ void act_rows_kernel(const IT* __restrict__ z, int nsplit, size_t spl
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= n) return;
     const float v = load_parts_t(z, i, nsplit, split_stride);
-    float a;
-    if (act == ACT_RELU2) { a = fmaxf(v, 0.f); a *= a; }
-    else if (act == ACT_SILU) a = v * sigmoidf(v);
-    else if (act == ACT_GELU_TANH) a = gelu_tanhf(v);
-    else a = v;
-    out[i] = from_float<OT>(a);
-}
-
-__device__ __forceinline__ float act_of(float v, int act) {
-    if (act == ACT_RELU2) { const float a = fmaxf(v, 0.f); return a * a; }
-    if (act == ACT_SILU) return v * sigmoidf(v);
-    if (act == ACT_GELU_TANH) return gelu_tanhf(v);
-    return v;
+    out[i] = from_float<OT>(act_of(v, act));
 }
 
 // four elements per thread (n % 4 == 0, 16-byte aligned, parts a multiple of four elements apart)
@@ -211,8 +208,9 @@ __global__ void gated_rmsnorm_kernel(const float* __restrict__ o, const float* _
 
 // ---- q/k norm over the whole projection, rotation, append ------------------------------------------
 // A row of the product holds [q: nq * dk | k: nkv * dk | v: nkv * dv | anything else]; a layer that
-// reads another layer's cache has [q | anything else] and has_kv = 0.  One page of the cache holds
-// [keys: nkv][P][dk] followed by [values: nkv][P][dv].
+// reads another layer's cache has [q | anything else] and has_kv = 0.  With v_from_k the row holds [q | k | anything
+// else] and the values are the keys as projected (with their bias, before norm and rotation; dv = dk).  One page of the
+// cache holds [keys: nkv][P][dk] followed by [values: nkv][P][dv].
 template <typename QT, typename CT>
 __global__ void qknorm_rope_append_kernel(const float* __restrict__ qkv, int nsplit, size_t split_stride, int ld,
                                           const float* __restrict__ q_weight, const float* __restrict__ k_weight,
@@ -222,7 +220,8 @@ __global__ void qknorm_rope_append_kernel(const float* __restrict__ qkv, int nsp
                                           QT* __restrict__ q_out, CT* __restrict__ cache, int nq, int nkv, int dk,
                                           int dv, int P, int num_pages, int has_kv, int* __restrict__ status,
                                           int per_head, float v_eps, size_t page_extra, float temp_coef,
-                                          double temp_every, float v_scale) {
+                                          double temp_every, float v_scale, const float* __restrict__ bias,
+                                          int v_from_k) {
     extern __shared__ float sh[];            // q row, k row, cos, sin (and the v row, if it is normalised)
     __shared__ float scratch[33];
     pdl_launch_dependents();
@@ -236,11 +235,16 @@ __global__ void qknorm_rope_append_kernel(const float* __restrict__ qkv, int nsp
     float* cs = ks + kw;
     float* sn = cs + rhalf;
     const size_t base = (size_t)t * ld;
+    float* vs = sn + rhalf;                  // [vw], only with v_eps > 0 or v_from_k
     float ssq = 0.f, ssk = 0.f;
     for (int i = threadIdx.x; i < qw + kw; i += blockDim.x) {
-        const float v = load_parts(qkv, base + i, nsplit, split_stride);
+        const float v = load_parts(qkv, base + i, nsplit, split_stride) + (bias ? bias[i] : 0.f);
         sh[i] = v;
-        if (i < qw) ssq += v * v; else ssk += v * v;
+        if (i < qw) ssq += v * v;
+        else {
+            ssk += v * v;
+            if (v_from_k) vs[i - qw] = v;
+        }
     }
     for (int i = threadIdx.x; i < rhalf; i += blockDim.x) {
         float s, c;
@@ -248,8 +252,7 @@ __global__ void qknorm_rope_append_kernel(const float* __restrict__ qkv, int nsp
         cs[i] = c;
         sn[i] = s;
     }
-    float* vs = sn + rhalf;                  // [vw], only with v_eps > 0
-    if (v_eps > 0.f)
+    if (v_eps > 0.f && !v_from_k)
         for (int i = threadIdx.x; i < vw; i += blockDim.x) vs[i] = load_parts(qkv, base + qw + kw + i, nsplit, split_stride);
     if (per_head) {
         // one norm per head over its dk elements, the weight [dk] shared by the heads: a warp per head; and a temperature
@@ -323,7 +326,7 @@ __global__ void qknorm_rope_append_kernel(const float* __restrict__ qkv, int nsp
         for (int i = threadIdx.x; i < vw; i += blockDim.x) {
             const int g = i / dv, e = i - g * dv;
             page_v[((size_t)g * P + within) * dv + e] =
-                from_float<CT>(v_scale * (v_eps > 0.f ? vs[i] : load_parts(qkv, base + qw + kw + i, nsplit, split_stride)));
+                from_float<CT>(v_scale * (v_eps > 0.f || v_from_k ? vs[i] : load_parts(qkv, base + qw + kw + i, nsplit, split_stride)));
         }
     }
 }
@@ -377,7 +380,7 @@ MHB_EXPORT int mhb_norm_mix(float* x, const void* delta, int delta_dtype, int ns
 MHB_EXPORT int mhb_act_rows(const void* z, int in_dtype, int nsplit, long long split_stride, void* out,
                             int out_dtype, long long n, int act, cudaStream_t stream) {
     if (n <= 0) return 0;
-    if (act < 0 || act > ACT_COPY) return fail("act_rows: unknown activation %d", act);
+    if (act < 0 || act > ACT_GELU) return fail("act_rows: unknown activation %d", act);
     if (nsplit > 1 && in_dtype != MHB_F32) return fail("act_rows: split partials must be float32");
     const int threads = 256;
     if (n % 4 == 0 && !((uintptr_t)z & 15) && !((uintptr_t)out & 15) && split_stride % 4 == 0) {
@@ -423,28 +426,31 @@ MHB_EXPORT int mhb_gated_rmsnorm(const float* o, const float* gate, int gate_nsp
 // projections.  v_eps > 0: every head's value is divided by its root mean square (with that eps) before it is stored.
 // page_extra: elements of a page behind its keys and values (left alone here).  temp_coef != 0 (with per_head): q is
 // multiplied by 1 + temp_coef ln(floor((position + 1) / temp_every) + 1).  v_scale: a factor on the stored values.
-// With per_head the weights may be null (norms without a weight).
+// With per_head the weights may be null (norms without a weight).  bias (or null): [nq dk + nkv dk], added to q and k
+// before anything else.  v_from_k: the row has no v columns, the values are the keys as projected.
 MHB_EXPORT int mhb_qknorm_rope_append_opts(const float* qkv, int nsplit, long long split_stride, int ld,
                                       const float* q_weight, const float* k_weight, float eps, const int* positions,
                                       const int* tok_seg, const int* block_table, int table_width,
                                       const float* inv_freq, int rdim, void* q_out, void* cache, int dtype, int T,
                                       int nq, int nkv, int dk, int dv, int P, int num_pages, int has_kv, int* status,
                                       int per_head, float v_eps, long long page_extra, float temp_coef,
-                                      double temp_every, float v_scale, cudaStream_t stream) {
+                                      double temp_every, float v_scale, const float* bias, int v_from_k,
+                                      cudaStream_t stream) {
     if (T <= 0) return 0;
+    if (v_from_k && (dv != dk || !has_kv)) return fail("qknorm_rope_append: keys that serve as values are as wide as these");
     if (!per_head && (!q_weight || (has_kv && !k_weight) || temp_coef != 0.f))
         return fail("qknorm_rope_append: norms over whole projections have weights and no temperature");
     if (temp_coef != 0.f && !(temp_every > 0.)) return fail("qknorm_rope_append: a temperature needs a positive step");
     if (rdim < 0 || rdim > dk || (rdim & 1)) return fail("qknorm_rope_append: %d rotated elements of a head of %d", rdim, dk);
     const int qw = nq * dk, kw = has_kv ? nkv * dk : 0;
-    const size_t smem = sizeof(float) * ((size_t)qw + kw + rdim + (v_eps > 0.f && has_kv ? (size_t)nkv * dv : 0));
+    const size_t smem = sizeof(float) * ((size_t)qw + kw + rdim + ((v_eps > 0.f || v_from_k) && has_kv ? (size_t)nkv * dv : 0));
     MHB_DISPATCH_DTYPE(dtype, CT, {
         auto kern = qknorm_rope_append_kernel<CT, CT>;
         if (allow_smem(kern, smem, "qknorm_rope_append")) return -1;
         launch_kernel(kern, dim3(T), dim3(row_threads(qw + kw)), smem, stream, qkv, nsplit, (size_t)split_stride, ld,
                       q_weight, k_weight, eps, positions, tok_seg, block_table, table_width, inv_freq, rdim,
                       (CT*)q_out, (CT*)cache, nq, nkv, dk, dv, P, num_pages, has_kv, status, per_head, v_eps,
-                      (size_t)page_extra, temp_coef, temp_every, v_scale);
+                      (size_t)page_extra, temp_coef, temp_every, v_scale, bias, v_from_k);
     });
     return check_launch("qknorm_rope_append");
 }
@@ -457,5 +463,5 @@ MHB_EXPORT int mhb_qknorm_rope_append(const float* qkv, int nsplit, long long sp
                                       cudaStream_t stream) {
     return mhb_qknorm_rope_append_opts(qkv, nsplit, split_stride, ld, q_weight, k_weight, eps, positions, tok_seg,
                                        block_table, table_width, inv_freq, rdim, q_out, cache, dtype, T, nq, nkv, dk, dv,
-                                       P, num_pages, has_kv, status, 0, 0.f, 0, 0.f, 1., 1.f, stream);
+                                       P, num_pages, has_kv, status, 0, 0.f, 0, 0.f, 1., 1.f, nullptr, 0, stream);
 }

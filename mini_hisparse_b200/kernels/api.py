@@ -97,6 +97,14 @@ def embed(table, tokens, out, status=None, scale: float = 1.0, copy=None):
                                      _ptr(copy), _stream()), "embed")
 
 
+def embed_norm(table, weight, eps, tokens, out, status=None):
+    """out[t] = rms(table[tokens[t]]) * weight as float32; ids outside the table give zeros and set status bit 0."""
+    lib = build.load("elementwise")
+    T, H = out.shape
+    _check(lib, lib.mhb_embed_norm(_ptr(table), c_int(dtype_code(table.dtype)), _ptr(tokens), _ptr(weight), c_float(eps),
+                                   _ptr(out), c_int(T), c_int(H), c_int(table.shape[0]), _ptr(status), _stream()), "embed_norm")
+
+
 def norm_mix(x, weight, eps, *, delta=None, nsplit=1, split_stride=0, alpha=1.0, keep=0.0, copy=None):
     """x <- keep * x + rms(alpha * x + delta) * weight, row by row in float32, in place; ``copy`` (compute
     dtype, same shape) receives the new rows too.  alpha = 0 leaves x out of the norm (a normalised branch
@@ -115,13 +123,13 @@ def norm_mix(x, weight, eps, *, delta=None, nsplit=1, split_stride=0, alpha=1.0,
                                  c_int(R), c_int(H), _stream()), "norm_mix")
 
 
-ACTIVATIONS = {"relu2": 0, "silu": 1, "gelu_tanh": 2, "copy": 3}
+ACTIVATIONS = {"relu2": 0, "silu": 1, "gelu_tanh": 2, "copy": 3, "gelu": 4}
 GLU_ACTS = {"silu": 0, "gelu_tanh": 1}          # activations of a gated feed-forward's gate
 
 
 def act_rows(z, out, act: str, nsplit=1, split_stride=0):
     """out = act(z) element by element in float32; z may be split-K parts.  act: relu2 (the square of
-    relu), silu, gelu_tanh, copy (a conversion only)."""
+    relu), silu, gelu_tanh, gelu (the exact one, with the error function), copy (a conversion only)."""
     lib = build.load("postnorm")
     if act not in ACTIVATIONS:
         raise KernelError(f"act_rows: unknown activation {act!r}; known: {sorted(ACTIVATIONS)}")
@@ -166,7 +174,7 @@ def gated_rmsnorm(o, weight, eps, out, gate=None, gate_nsplit=1, gate_split_stri
 
 def qknorm_rope_append(qkv, q_weight, k_weight, eps, positions, tok_seg, block_table, inv_freq, rotary_dim, q_out,
                        cache, *, nq, nkv, dk, dv, page_size, has_kv=True, nsplit=1, split_stride=0, status=None,
-                       per_head=False, v_eps=0.0, page_extra=0, q_temp=None, v_scale=1.0):
+                       per_head=False, v_eps=0.0, page_extra=0, q_temp=None, v_scale=1.0, bias=None, v_from_k=False):
     """RMS norm over the whole q projection and over the whole k projection, rotation of the first
     ``rotary_dim`` elements of every head (pairs (i, i + rotary_dim/2)), q to ``q_out`` [T, nq dk], k and v
     into the pages of ``cache`` (one layer's pool; a page holds [nkv][P][dk] keys then [nkv][P][dv] values).
@@ -175,7 +183,9 @@ def qknorm_rope_append(qkv, q_weight, k_weight, eps, positions, tok_seg, block_t
     heads.  ``v_eps`` > 0: every head's value is divided by its root mean square before it is stored.
     ``page_extra``: elements of a page behind its keys and values, which this kernel leaves alone.  With ``per_head``
     the weights may be None, and ``q_temp`` = (coef, every) multiplies q by
-    1 + coef ln(floor((position + 1) / every) + 1).  ``v_scale``: a factor on the stored values."""
+    1 + coef ln(floor((position + 1) / every) + 1).  ``v_scale``: a factor on the stored values.  ``bias`` float32
+    [nq dk + nkv dk] is added to q and k first; with ``v_from_k`` a row is [q | k | ...] and the values are the keys as
+    projected (with the bias, before norm and rotation)."""
     lib = build.load("postnorm")
     T = q_out.shape[0]
     if qkv.dtype != torch.float32 or qkv.stride(-1) != 1:
@@ -191,7 +201,7 @@ def qknorm_rope_append(qkv, q_weight, k_weight, eps, positions, tok_seg, block_t
         c_int(T), c_int(nq), c_int(nkv), c_int(dk), c_int(dv), c_int(page_size),
         c_int(cache.shape[0] if has_kv else 0), c_int(1 if has_kv else 0), _ptr(status), c_int(1 if per_head else 0),
         c_float(v_eps or 0.0), c_longlong(page_extra), c_float(q_temp[0] if q_temp else 0.0),
-        c_double(q_temp[1] if q_temp else 1.0), c_float(v_scale), _stream()),
+        c_double(q_temp[1] if q_temp else 1.0), c_float(v_scale), _ptr(bias), c_int(1 if v_from_k else 0), _stream()),
         "qknorm_rope_append")
 
 
@@ -415,7 +425,7 @@ def gemm_tc_glu(a, w, out, act: str, *, swap: bool, bn: int, status=None, scratc
         "gemm_tc_glu")
 
 
-PRODUCT_ACTS = ("gelu_tanh",)       # activations that the tensor-core product's epilogue takes without a gate
+PRODUCT_ACTS = {"gelu_tanh": 1, "gelu": 2, "relu2": 3}       # activations that the tensor-core product's epilogue takes without a gate
 
 
 def gemm_tc_act(a, w, out, act: str, *, status=None, scratch=None):
@@ -432,7 +442,7 @@ def gemm_tc_act(a, w, out, act: str, *, status=None, scratch=None):
         raise KernelError("gemm_tc_act: the last dimension must be contiguous")
     _check(lib, lib.mhb_gemm_tc_act(
         _ptr(a), _ptr(w), _ptr(out), c_int(M), c_int(N), c_int(K), c_longlong(a.stride(0)), c_longlong(w.stride(0)),
-        c_longlong(out.stride(0)), *_scratch_ptrs(scratch), _ptr(status), c_int(GLU_ACTS[act]), _stream()), "gemm_tc_act")
+        c_longlong(out.stride(0)), *_scratch_ptrs(scratch), _ptr(status), c_int(PRODUCT_ACTS[act]), _stream()), "gemm_tc_act")
 
 
 def rope_table(positions, inv_freq, table):
@@ -477,7 +487,8 @@ def gemm_tc_qkv_rope(x, w, bias, cos_sin, positions, tok_seg, block_table, q_out
 def attention_simt(q, cache, out, part_acc, part_ml, items, num_items, max_items, positions,
                    block_table, tok_part_row, *, nq, nkv, d, page_size, window=0, scale=None, dv=None,
                    sink=None, gate=None, gate_nsplit=1, gate_split_stride=0, kparts=1, softcap=0.0,
-                   shared_kv=False, gate_per_head=False, keep_first=0, pool=0, all_values=False, value_head=None):
+                   shared_kv=False, gate_per_head=False, keep_first=0, pool=0, all_values=False, value_head=None,
+                   slopes=None):
     """CUDA-core attention over the items of a plan.  Options: ``dv`` values of another width than the
     keys (a page then holds the keys of all KV heads followed by their values), ``sink`` float32 [nq]
     (one extra term exp(sink_h) in the softmax's denominator), ``gate`` (the output is multiplied by its
@@ -488,14 +499,15 @@ def attention_simt(q, cache, out, part_acc, part_ml, items, num_items, max_items
     start of a sequence stay visible, or (``pool``) every block of ``pool`` positions that the window has passed
     wholly is seen as one key and value, its means, from the tail of its page (csrc/maskparts.cu).
     ``all_values``: every query head's weights are applied to the values of all KV heads, and ``out`` is
-    [T, nq, nkv * dv]; ``value_head``: to the values of that one KV head."""
+    [T, nq, nkv * dv]; ``value_head``: to the values of that one KV head.  ``slopes`` float32 [nq]: slope_h times the
+    distance of query and key is taken off the scaled score."""
     lib = build.load("attention_simt")
     if scale is None:
         scale = float(d) ** -0.5
     if keep_first or pool or all_values or value_head is not None:
         if keep_first and pool:
             raise KernelError("attention: kept first positions or pooled blocks, not both")
-        if kparts != 1 or softcap or shared_kv or gate_per_head:
+        if kparts != 1 or softcap or shared_kv or gate_per_head or slopes is not None:
             raise KernelError("attention: keys beyond the window go with plain keys and values only")
         g = _gate_args(gate, gate_nsplit, gate_split_stride)
         _check(lib, lib.mhb_attention_simt_masked(
@@ -507,7 +519,7 @@ def attention_simt(q, cache, out, part_acc, part_ml, items, num_items, max_items
             c_int(1 if keep_first else 2 if pool else 0), c_int(keep_first or pool or 0),
             c_int(1 if all_values else 0 if value_head is None else 2 + value_head), _stream()), "attention")
         return
-    general = kparts != 1 or softcap or shared_kv or gate_per_head or out.dtype != q.dtype
+    general = kparts != 1 or softcap or shared_kv or gate_per_head or out.dtype != q.dtype or slopes is not None
     if dv is not None or sink is not None or gate is not None or general:
         g = _gate_args(gate, gate_nsplit, gate_split_stride)
         _check(lib, lib.mhb_attention_simt_ext(
@@ -516,7 +528,7 @@ def attention_simt(q, cache, out, part_acc, part_ml, items, num_items, max_items
             c_int(block_table.shape[-1]), _ptr(tok_part_row), c_int(nq), c_int(nkv), c_int(d), c_int(dv or d),
             c_int(page_size), c_int(cache.shape[0]), c_int(window or 0), c_float(scale), _ptr(sink),
             g[0], g[1], g[2], g[3], c_int(kparts), c_float(softcap or 0.0), c_int(1 if shared_kv else 0),
-            c_int(1 if gate_per_head else 0), c_int(1 if out.dtype == torch.float32 else 0), _stream()),
+            c_int(1 if gate_per_head else 0), c_int(1 if out.dtype == torch.float32 else 0), _ptr(slopes), _stream()),
             "attention")
         return
     _check(lib, lib.mhb_attention_simt(
@@ -582,11 +594,11 @@ def attention_mma_ext_supports(d: int, dv: int) -> bool:
 def attention_mma_ext(q, cache, out, part_acc, part_ml, items, num_items, rows, positions, block_table,
                       tok_part_row, *, nq, nkv, d, dv, page_size, window=0, scale=None, tok_nsplit=None,
                       counters=None, sink=None, gate=None, gate_nsplit=1, gate_split_stride=0, kparts=1, softcap=0.0,
-                      shared_kv=False, gate_per_head=False, keep_first=0, pool=0, value_head=None):
+                      shared_kv=False, gate_per_head=False, keep_first=0, pool=0, value_head=None, slopes=None):
     """attention_mma with the options of attention_simt: values ``dv`` wide in pages that hold the keys of
     all KV heads followed by their values, a ``sink`` per query head, a ``gate`` on the output; the softmax's
     weights enter the value product as two bfloat16 numbers each (16 bits instead of 8).  ``kparts``,
-    ``softcap``, ``shared_kv``, ``gate_per_head``, ``keep_first`` and ``pool`` as in attention_simt; ``out`` may be
+    ``softcap``, ``shared_kv``, ``gate_per_head``, ``keep_first``, ``pool`` and ``slopes`` as in attention_simt; ``out`` may be
     float32.  ``value_head``: every query head's weights are applied to the values of that one KV head; "all": to
     the values of every KV head in turn in one launch, ``out`` being [nkv, T, nq, dv] (a plane per KV head), the partial
     buffers [nkv, rows, nq, ...] and the counters [nkv, ...] likewise (for a mixer that mixes the heads' weights)."""
@@ -601,7 +613,7 @@ def attention_mma_ext(q, cache, out, part_acc, part_ml, items, num_items, rows, 
     if keep_first or pool or value_head is not None:
         if keep_first and pool:
             raise KernelError("attention: kept first positions or pooled blocks, not both")
-        if kparts != 1 or softcap or shared_kv or gate_per_head or sink is not None:
+        if kparts != 1 or softcap or shared_kv or gate_per_head or sink is not None or slopes is not None:
             raise KernelError("attention: keys beyond the window go with plain keys and values only")
         planes = (0, 0, 0)
         if value_head == "all":
@@ -627,7 +639,7 @@ def attention_mma_ext(q, cache, out, part_acc, part_ml, items, num_items, rows, 
         _ptr(tok_part_row), _ptr(tok_nsplit), _ptr(counters), c_int(nq), c_int(nkv), c_int(d), c_int(dv),
         c_int(page_size), c_int(cache.shape[0]), c_int(window or 0), c_float(scale), _ptr(sink),
         g[0], g[1], g[2], g[3], c_int(kparts), c_float(softcap or 0.0), c_int(1 if shared_kv else 0),
-        c_int(1 if gate_per_head else 0), c_int(1 if out.dtype == torch.float32 else 0), _stream()),
+        c_int(1 if gate_per_head else 0), c_int(1 if out.dtype == torch.float32 else 0), _ptr(slopes), _stream()),
         "attention_mma_ext")
 
 
@@ -740,11 +752,11 @@ def attention_tc(q, cache, out, items, num_items, positions, block_table, *, nq,
 def attention_tma_ext(q, cache, out, part_acc, part_ml, items, num_items, rows, positions, block_table,
                       tok_part_row, *, nq, nkv, d, page_size, window=0, scale=None, tok_nsplit=None,
                       counters=None, status=None, fresh=0, sink=None, gate=None, gate_nsplit=1, gate_split_stride=0,
-                      gate_per_head=False, shared_kv=False, softcap=0.0):
+                      gate_per_head=False, shared_kv=False, softcap=0.0, slopes=None):
     """attention_tma with a ``sink`` per query head, a ``gate`` on the output (``gate_per_head``: one column per
     head) and softmax weights that keep 16 bits in the value product; keys and values are both ``d`` wide.
     ``shared_kv``: the pool is [pages, P, d] and a row is its position's key and value at once; ``softcap`` caps
-    the scaled scores; ``out`` may be float32."""
+    the scaled scores; ``slopes`` as in attention_simt; ``out`` may be float32."""
     lib = build.load("attention_tma")
     if q.dtype != torch.bfloat16 or cache.dtype != torch.bfloat16 or not cache.is_contiguous():
         raise KernelError("attention_tma_ext: q and the (contiguous) pool must be bfloat16")
@@ -757,18 +769,18 @@ def attention_tma_ext(q, cache, out, part_acc, part_ml, items, num_items, rows, 
         _ptr(tok_part_row), _ptr(tok_nsplit), _ptr(counters), c_int(nq), c_int(nkv), c_int(d),
         c_int(page_size), c_int(cache.shape[0]), c_int(window or 0), c_int(fresh), c_float(scale), _ptr(sink),
         g[0], g[1], g[2], g[3], c_int(1 if gate_per_head else 0), c_int(1 if shared_kv else 0),
-        c_float(softcap or 0.0), c_int(1 if out.dtype == torch.float32 else 0), _ptr(status), _stream()),
+        c_float(softcap or 0.0), c_int(1 if out.dtype == torch.float32 else 0), _ptr(slopes), _ptr(status), _stream()),
         "attention_tma_ext")
 
 
 def attention_tc_ext(q, cache, out, items, num_items, positions, block_table, *, nq, nkv, d, page_size,
                      window=0, scale=None, status=None, part_acc=None, part_ml=None, tok_part_row=None,
                      sink=None, gate=None, gate_nsplit=1, gate_split_stride=0, gate_per_head=False, shared_kv=False,
-                     softcap=0.0):
+                     softcap=0.0, slopes=None):
     """attention_tc with a ``sink`` per query head, a ``gate`` on the output (``gate_per_head``: one column
     per head) and softmax weights that keep 16 bits in the value product; keys and values are both ``d``
     wide.  ``shared_kv``: the pool is [pages, P, d] and a row is its position's key and value at once;
-    ``softcap`` caps the scaled scores; ``out`` may be float32."""
+    ``softcap`` caps the scaled scores; ``slopes`` as in attention_simt; ``out`` may be float32."""
     lib = build.load("attention_tc")
     if q.dtype != torch.bfloat16 or cache.dtype != torch.bfloat16 or not cache.is_contiguous():
         raise KernelError("attention_tc_ext: q and the (contiguous) pool must be bfloat16")
@@ -781,7 +793,7 @@ def attention_tc_ext(q, cache, out, items, num_items, positions, block_table, *,
         c_int(nq), c_int(nkv), c_int(d), c_int(page_size), c_int(cache.shape[0]), c_int(window or 0),
         c_float(scale), _ptr(sink), g[0], g[1], g[2], g[3], c_int(1 if gate_per_head else 0),
         c_int(1 if shared_kv else 0), c_float(softcap or 0.0), c_int(1 if out.dtype == torch.float32 else 0),
-        _ptr(status), _stream()), "attention_tc_ext")
+        _ptr(slopes), _ptr(status), _stream()), "attention_tc_ext")
 
 
 def attention_combine(part_acc, part_ml, tok_part_row, tok_nsplit, out, *, nq, d, every=0, gate=None,
@@ -1097,18 +1109,22 @@ def moe_plan_words(pairs: int, experts: int) -> int:
     return 1 + 3 * moe_max_tiles(pairs, experts) + 2 * pairs
 
 
-def moe_route(logits, correction, chosen, weights, *, outputs, top, groups=1, keep=1, bias=None):
+def moe_route(logits, correction, chosen, weights, *, outputs, top, groups=1, keep=1, bias=None, score="softmax",
+              group_two=False, normalise=True, factor=1.0):
     """Per token: softmax over the first ``outputs`` columns of the float32 Product ``logits`` (plus ``bias``, if
     there is one), choice by softmax + correction (None: none) inside the best ``keep`` of ``groups`` groups,
     ``chosen`` int32 [T, top] and the chosen outputs' softmax values divided by their sum as ``weights`` float32
     [T, top]: without a correction that is the choice of the largest logits, weighted by the softmax over the
-    chosen logits alone."""
+    chosen logits alone.  ``score`` "sigmoid": the sigmoid of every output instead of the softmax; ``group_two``: a group's
+    score is the sum of its two largest choice scores; ``normalise`` False: the weights are not divided by their sum;
+    ``factor`` multiplies them."""
     lib = build.load("moe")
     T = chosen.shape[0]
-    _check(lib, lib.mhb_moe_route_biased(*_parts_args(logits.tensor, logits.nsplit, logits.split_stride),
-                                         c_int(logits.tensor.stride(-2)), _ptr(bias), _ptr(correction), _ptr(chosen),
-                                         _ptr(weights), c_int(T), c_int(outputs), c_int(top), c_int(groups),
-                                         c_int(keep), _stream()), "moe_route")
+    _check(lib, lib.mhb_moe_route_opts(*_parts_args(logits.tensor, logits.nsplit, logits.split_stride),
+                                       c_int(logits.tensor.stride(-2)), _ptr(bias), _ptr(correction), _ptr(chosen),
+                                       _ptr(weights), c_int(T), c_int(outputs), c_int(top), c_int(groups), c_int(keep),
+                                       c_int({"softmax": 0, "sigmoid": 1}[score]), c_int(1 if group_two else 0),
+                                       c_int(1 if normalise else 0), c_float(factor), _stream()), "moe_route")
 
 
 def moe_plan(chosen, plan, *, experts):
@@ -1123,24 +1139,29 @@ def moe_plan(chosen, plan, *, experts):
                                  c_int(moe_max_tiles(pairs, experts)), _ptr(plan), _stream()), "moe_plan")
 
 
-def moe_linear(x, plan, w, out, *, pairs, experts, gather: bool, glu: bool):
+MOE_ACTS = {None: 0, "silu_glu": 1, "relu2": 2}        # what moe_linear does to its sums
+
+
+def moe_linear(x, plan, w, out, *, pairs, experts, gather: bool, act: str | None = None):
     """out[r] = w[expert of row r] applied to x[token of row r] (``gather``) or to x[r]; ``w`` [experts, N, K], or
-    [experts, 2 N, K] holding gate above up with ``glu`` (then out = silu(gate x) * (up x)); float32 accumulation."""
+    [experts, 2 N, K] holding gate above up with ``act`` "silu_glu" (then out = silu(gate x) * (up x)); ``act`` "relu2":
+    the square of relu; float32 accumulation."""
     lib = build.load("moe")
     N, Kd = out.shape[1], x.shape[1]
-    if w.dtype != x.dtype or tuple(w.shape) != (experts, (2 if glu else 1) * N, Kd) or not w.is_contiguous():
+    if w.dtype != x.dtype or tuple(w.shape) != (experts, (2 if act == "silu_glu" else 1) * N, Kd) or not w.is_contiguous():
         raise KernelError(f"moe_linear: weights {list(w.shape)} for rows {Kd} wide and outputs {N} wide")
     if x.stride(1) != 1 or not out.is_contiguous():
         raise KernelError("moe_linear: contiguous rows")
     _check(lib, lib.mhb_moe_linear(_ptr(x), c_int(dtype_code(x.dtype)), c_longlong(x.stride(0)), _ptr(plan),
                                    c_int(moe_max_tiles(pairs, experts)), c_int(pairs), c_int(1 if gather else 0), _ptr(w),
-                                   _ptr(out), c_int(dtype_code(out.dtype)), c_int(N), c_int(Kd), c_int(1 if glu else 0),
+                                   _ptr(out), c_int(dtype_code(out.dtype)), c_int(N), c_int(Kd), c_int(MOE_ACTS[act]),
                                    _stream()), "moe_linear")
 
 
 def moe_combine(y, plan, chosen, weights, h, out, *, experts, shared=None, shared_gate=None):
     """out[t] = sum_k weights[t, k] * (y[row of pair (t, k)], or h[t] for an identity expert) + sigmoid(shared_gate[t])
-    * shared[t]; ``shared`` and ``shared_gate`` are float32 Products (the gate one column)."""
+    * shared[t]; ``shared`` and ``shared_gate`` are float32 Products (the gate one column; without it shared[t] is added as
+    it is)."""
     lib = build.load("moe")
     T, top = chosen.shape
     pairs = T * top
@@ -1152,6 +1173,7 @@ def moe_combine(y, plan, chosen, weights, h, out, *, experts, shared=None, share
     g_ld = 0
     if shared is not None:
         sh = _parts_args(shared.tensor, shared.nsplit, shared.split_stride)
+    if shared_gate is not None:
         sg = _parts_args(shared_gate.tensor, shared_gate.nsplit, shared_gate.split_stride)
         g_ld = shared_gate.tensor.stride(-2)
     _check(lib, lib.mhb_moe_combine(_ptr(y), _ptr(plan), c_int(moe_max_tiles(pairs, experts)), c_int(pairs), _ptr(chosen),
@@ -1245,6 +1267,33 @@ def delta_scan(q, k, v, beta, decay, state, out, tok_seg, seg_slot, positions, *
                                    c_longlong(state.stride(0)), _ptr(out), _ptr(tok_seg), _ptr(seg_slot), _ptr(positions),
                                    c_int(T), c_int(S), c_int(heads), c_int(kv_heads), c_int(dk), c_int(dv),
                                    c_int(1 if writable else 0), _stream()), "delta_scan")
+
+
+# ---- convolved heads of attention (csrc/headconv.cu) ----
+def head_conv_append(proj, taps, q_weight, k_weight, eps, keep, ctx, block_table, q_out, cache, *, nq, nkv, dk, dv,
+                     page_size, has_kv=True, q_temp=None):
+    """Columns [q: nq dk | k: nkv dk | v: nkv dv] of the float32 Product ``proj`` (with ``has_kv`` False [q] alone) through
+    a short causal convolution per channel over time (``taps`` float32 [taps, channels], no activation); q and k
+    RMS-normalised head by head (weights [dk] shared by the heads, or None); q times 1 + coef ln(floor((position + 1) /
+    every) + 1) for ``q_temp`` = (coef, every); q to ``q_out`` [T, nq dk], k and v into the pages of ``cache``.  ``keep``
+    float32 [slots, taps - 1, channels]: a slot's last projected rows, read and renewed."""
+    lib = build.load("headconv")
+    T = q_out.shape[0]
+    ntaps, C = _taps(taps, "head_conv_append")
+    if C != nq * dk + (nkv * (dk + dv) if has_kv else 0):
+        raise KernelError(f"head_conv_append: filters for {C} channels")
+    if proj.tensor.dtype != torch.float32 or not q_out.is_contiguous():
+        raise KernelError("head_conv_append: the product is float32, q contiguous")
+    if has_kv and (cache is None or cache.dtype != q_out.dtype or not cache.is_contiguous()):
+        raise KernelError("head_conv_append: the pool must be contiguous and of the activations' dtype")
+    _check(lib, lib.mhb_head_conv_append(
+        *_parts_args(proj.tensor, proj.nsplit, proj.split_stride), c_int(proj.tensor.stride(-2)), _ptr(taps), c_int(ntaps),
+        _ptr(q_weight), _ptr(k_weight), c_float(eps), *_keep_args(keep, ntaps - 1, C, "head_conv_append"), *_seg_args(ctx),
+        _ptr(block_table), c_int(block_table.shape[-1]), _ptr(q_out), _ptr(cache if has_kv else None),
+        c_int(dtype_code(q_out.dtype)), c_int(T), c_int(len(ctx.segments)), c_int(ctx.longest), c_int(nq), c_int(nkv),
+        c_int(dk), c_int(dv), c_int(page_size), c_int(cache.shape[0] if has_kv else 0), c_int(1 if has_kv else 0),
+        c_float(q_temp[0] if q_temp else 0.0), c_double(q_temp[1] if q_temp else 1.0), _ptr(ctx.status), _stream()),
+        "head_conv_append")
 
 
 # ---- convolutions over time and element-by-element recurrences (csrc/timeconv.cu, selscan.cu) ----

@@ -12,6 +12,7 @@ from .spec import LayerSpec, StateNeed
 @register_block("pre_norm")
 class PreNormBlock(Block):
     """x = x + mixer(norm1(x)); x = x + ff(norm2(x))   (mini_hisparse/model.py:137,155-158).
+    A layer without the roles "ff_norm" and "feed_forward" has the first half only.
 
     The residual adds are folded into the norms that follow them: the block receives the
     previous block's still-unadded output as ``pending`` and returns its own.
@@ -21,20 +22,22 @@ class PreNormBlock(Block):
         self.spec = spec
         self.mixer_norm = NORMS.build(spec.part("mixer_norm"), rt=rt)
         self.mixer = MIXERS.build(spec.part("mixer"), rt=rt)
-        self.ff_norm = NORMS.build(spec.part("ff_norm"), rt=rt)
-        self.feed_forward = FEED_FORWARDS.build(spec.part("feed_forward"), rt=rt)
+        self.ff_norm = self.feed_forward = None
+        if spec.has("feed_forward"):
+            self.ff_norm = NORMS.build(spec.part("ff_norm"), rt=rt)
+            self.feed_forward = FEED_FORWARDS.build(spec.part("feed_forward"), rt=rt)
 
     def parts(self):
-        return {
-            "mixer_norm": self.mixer_norm,
-            "mixer": self.mixer,
-            "ff_norm": self.ff_norm,
-            "feed_forward": self.feed_forward,
-        }
+        out = {"mixer_norm": self.mixer_norm, "mixer": self.mixer}
+        if self.feed_forward is not None:
+            out.update(ff_norm=self.ff_norm, feed_forward=self.feed_forward)
+        return out
 
     def forward(self, x, pending: Product | None, ctx: StepContext, cache: CacheView | None) -> Product:
         h = self.mixer_norm.forward(x, ctx, delta=pending)
-        a = self.mixer.forward(h, ctx, cache)
+        a = self.mixer.forward(h, ctx, cache.narrow("mixer.") if cache is not None and cache.sides else cache)
+        if self.feed_forward is None:
+            return a
         h = self.ff_norm.forward(x, ctx, delta=a)
         return self.feed_forward.forward(h, ctx)
 

@@ -17,26 +17,36 @@ class TokenEmbedding(Part):
     ctx.extras["x_copy"], for a first block that reads the stream without normalising it.  With
     ``keep`` = (name, row width, first column) the rows are also left, in the compute dtype, in those
     columns of a matrix ctx.extras[name] [T, row width], for a later part that reads the embedding
-    output again (the input of a pass over repeated layers)."""
+    output again (the input of a pass over repeated layers).  With ``norm`` = (tensor's local name, eps) the row
+    enters the stream as rms(row) * weight, in the gather's kernel (then without a scale and a copy)."""
 
     def __init__(self, spec: PartSpec, rt=None):
         super().__init__(spec, rt)
+        self.norm = spec.get("norm")
+        self.norm_weight = None
         self.vocab = int(spec["vocab_size"])
         self.width = int(spec["hidden_size"])
         self.scale = float(spec.get("scale", 1.0))
         self.copy = bool(spec.get("copy", False))
         self.keep = spec.get("keep")
         self.weight_name = spec.get("weight_name", "weight")
+        if self.norm and (self.scale != 1.0 or self.copy):
+            raise ValueError("an embedding that normalises its rows takes no scale and keeps no copy")
         self.weight = None
 
     def kernel_modules(self):
         return ("mixparts",) if self.keep else ()
 
     def parameters(self):
-        return {self.weight_name: ParamSpec((self.vocab, self.width))}
+        p = {self.weight_name: ParamSpec((self.vocab, self.width))}
+        if self.norm:
+            p[self.norm[0]] = ParamSpec((self.width,), role="vector", init=("normal", 1.0, 0.1))
+        return p
 
     def load(self, tensors):
         self.weight = tensors[self.weight_name].contiguous()
+        if self.norm:
+            self.norm_weight = tensors[self.norm[0]].contiguous()
 
     def forward(self, ctx: StepContext) -> torch.Tensor:
         x = self._forward(ctx)
@@ -50,6 +60,9 @@ class TokenEmbedding(Part):
     def _forward(self, ctx: StepContext) -> torch.Tensor:
         x = ctx.ws.get("residual", (ctx.T, self.width), torch.float32)
         copy = None
+        if self.norm:
+            K.embed_norm(self.weight, self.norm_weight, float(self.norm[1]), ctx.tokens, x, status=ctx.status)
+            return x
         if self.copy and ctx.rt.dtype != torch.float32:
             copy = ctx.ws.get("x_copy", (ctx.T, self.width), ctx.rt.dtype)
         K.embed(self.weight, ctx.tokens, x, status=ctx.status, scale=self.scale, copy=copy)

@@ -45,8 +45,8 @@ class SwiGLU(FeedForward):
 
 @register_feed_forward("mlp_act")
 class ActivatedMLP(FeedForward):
-    """down(act(up(x))), no gate, no biases; ``activation``: "relu2" (the square of relu), "silu" or
-    "gelu_tanh", computed in float32 on the product's float32 output, or "polynorm":
+    """down(act(up(x))), no gate, no biases; ``activation``: "relu2" (the square of relu), "silu",
+    "gelu_tanh" or "gelu" (the exact one), computed in float32 on the product's float32 output, or "polynorm":
     act(z) = a rms(z) + b rms(z^2) + c rms(z^3) + e with the powers taken element by element, each divided by its
     own root mean square over the token's ``intermediate_size`` values (``eps`` inside the root), and the four numbers
     (a, b, c, e) stored as the tensor ``coef_name`` (default "act").  Tensor names: ``up_name`` and

@@ -61,7 +61,7 @@ class SinkAttention(Mixer):
         (float32, and every other width)."""
         if self.rt is None or self.rt.dtype != torch.bfloat16 or not K.attention_mma_ext_supports(self.dk, self.dv):
             return "simt"
-        if not self.scale > 0.0:        # the tensor-core kernels keep the sink in the raw products' units, sink / scale
+        if not self.scale > 0.0:        # the tensor-core kernels keep sink and slopes in the raw products' units
             return "simt"
         if page_size is not None and self.dk == self.dv and K.attention_tma_supports(self.dk, page_size):
             return "tc"
@@ -120,7 +120,7 @@ class SinkAttention(Mixer):
         attn = self._attend(q, gate, ctx, cache, sink=self.sink)
         return rt.linear(attn, self.o_weight, ws, "mix_out", out_dtype=torch.float32)
 
-    def _attend(self, q, gate: dict, ctx: StepContext, cache: CacheView, sink=None) -> torch.Tensor:
+    def _attend(self, q, gate: dict, ctx: StepContext, cache: CacheView, sink=None, slopes=None) -> torch.Tensor:
         """The plan's items over the cache, the merge of key splits and the gate: [T, q_heads * vdim] in the compute dtype."""
         rt, ws, T = ctx.rt, ctx.ws, q.shape[0]
         meta = cache.meta
@@ -135,14 +135,14 @@ class SinkAttention(Mixer):
             args = (q, cache.storage, attn, part_acc, part_ml)
             tail = (ctx.positions, meta["block_table"], meta["tok_part_row"])
             common = dict(nq=self.nq, nkv=self.nkv, d=self.dk, dv=self.dv, page_size=cache.page_size,
-                          window=self.window or 0, scale=self.scale, sink=sink, **gate)
+                          window=self.window or 0, scale=self.scale, sink=sink, slopes=slopes, **gate)
             if n_small:          # decoded tokens and short portions: 16-row tiles, key splits merged by the last CTA
                 chunks = -(-(self.nq // self.nkv) // ROW_TILE)
                 counters = ws.get_zeroed("attn_counters", (T * self.nkv * chunks,), torch.int32)
                 if family == "tc":      # TMA-fed tiles (keys and values of one width, pages that divide 64)
                     K.attention_tma_ext(*args, meta["items"], n_small, 16, *tail, nq=self.nq, nkv=self.nkv, d=self.dk,
                                         page_size=cache.page_size, window=self.window or 0, scale=self.scale,
-                                        sink=sink, **gate, tok_nsplit=meta["tok_nsplit"], counters=counters,
+                                        sink=sink, slopes=slopes, **gate, tok_nsplit=meta["tok_nsplit"], counters=counters,
                                         status=ctx.status)
                 else:
                     K.attention_mma_ext(*args, meta["items"], n_small, 16, *tail, **common,
@@ -152,7 +152,8 @@ class SinkAttention(Mixer):
                 K.attention_tc_ext(q, cache.storage, attn, big_items, n_big, ctx.positions, meta["block_table"],
                                    nq=self.nq, nkv=self.nkv, d=self.dk, page_size=cache.page_size,
                                    window=self.window or 0, scale=self.scale, status=ctx.status, part_acc=part_acc,
-                                   part_ml=part_ml, tok_part_row=meta["tok_part_row"], sink=sink, **gate)
+                                   part_ml=part_ml, tok_part_row=meta["tok_part_row"], sink=sink, slopes=slopes,
+                                   **gate)
                 if meta.get("big_split"):
                     K.attention_combine(part_acc, part_ml, meta["tok_part_row"], meta["tok_nsplit"], attn,
                                         nq=self.nq, d=self.dv, **gate)
@@ -163,7 +164,7 @@ class SinkAttention(Mixer):
             K.attention_simt(q, cache.storage, attn, part_acc, part_ml, meta["items"], n, n, ctx.positions,
                              meta["block_table"], meta["tok_part_row"], nq=self.nq, nkv=self.nkv, d=self.dk,
                              dv=self.dv, page_size=cache.page_size, window=self.window or 0, scale=self.scale,
-                             sink=sink, **gate)
+                             sink=sink, slopes=slopes, **gate)
         if meta["any_split"]:
             K.attention_combine(part_acc, part_ml, meta["tok_part_row"], meta["tok_nsplit"], attn, nq=self.nq,
                                 d=self.dv, **gate)

@@ -423,9 +423,9 @@ def test_grouped_products_and_the_weighted_sum(dtype, E, identity, top, ff, W, s
     plan = torch.empty(K.moe_plan_words(pairs, E), dtype=torch.int32, device="cuda")
     K.moe_plan(cd, plan, experts=E)
     act = torch.full((pairs, ff), float("nan"), dtype=dtype, device="cuda")
-    K.moe_linear(hc, plan, gate_up.cuda(), act, pairs=pairs, experts=E, gather=True, glu=True)
+    K.moe_linear(hc, plan, gate_up.cuda(), act, pairs=pairs, experts=E, gather=True, act="silu_glu")
     y = torch.full((pairs, W), float("nan"), device="cuda")
-    K.moe_linear(act, plan, down.cuda(), y, pairs=pairs, experts=E, gather=False, glu=False)
+    K.moe_linear(act, plan, down.cuda(), y, pairs=pairs, experts=E, gather=False)
     out = torch.empty(T, W, device="cuda")
     K.moe_combine(y, plan, cd, wd, hc, out, experts=E, shared=sh, shared_gate=sg)
     close(out, ref, 1e-5 if dtype == torch.float32 else 0.01, "routed sum")
