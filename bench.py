@@ -17,10 +17,10 @@ of 128 to 4,096 tokens in portions of 512 beside decoding at the Qwen2.5-14B sha
 8,192 prompt tokens plus 512 generated ones at the Qwen2.5-32B shape with the page pool sized from
 free memory; tokens a second, step-time percentiles, roofline fractions, clocks, and the layer count.
 
-    python bench.py --workload koronex|dotivik|tudasun|rizovik|zetenex [--sizes 2k,4k]
+    python bench.py --workload koronex|dotivik|tudasun|rizovik|zetenex|rudutar [--sizes 2k,4k] [--beside MODEL]
 
-times a design beside the existing model that is closest to it (Koronex and Dotivik beside Qwen2 dense, Tudasun and
-Zetenex beside Koronex, Rizovik beside Tudasun) at equal width, heads, feed-forward width and layer
+times a design beside the existing model that is closest to it (Koronex and Dotivik beside Qwen2 dense, Tudasun,
+Zetenex and Rudutar beside Koronex, Rizovik beside Tudasun; --beside names another) at equal width, heads, feed-forward width and layer
 count (random weights): prefill of a 2,048-token prompt and decode at batch 8 with 4,096 tokens of context,
 each with its kernels' times, as one JSON line.
 """
@@ -39,6 +39,7 @@ sys.path.insert(0, str(ROOT))
 # Qwen2.5-7B shape, kept as data beside the package
 CONFIG_7B = json.loads((ROOT / "mini_hisparse_b200" / "configs" / "qwen2.5-7b-shape.json").read_text())
 WORKLOADS = {"serving14b": "qwen2.5-14b-shape.json", "long32b": "qwen2.5-32b-shape.json"}
+DESIGNS = ["koronex", "dotivik", "tudasun", "rizovik", "zetenex", "rudutar"]
 CONTEXT = 4096
 PREFILL_TOKENS = 2048
 PAGE = 16
@@ -70,8 +71,8 @@ def compare(args) -> int:
     from mini_hisparse_b200 import measure
 
     design = args.workload
-    result = measure.compare_architectures(tuple(args.sizes.split(",")), design=design, steps=args.steps,
-                                           warmup=args.warmup)
+    result = measure.compare_architectures(tuple(args.sizes.split(",")), design=design, beside=args.beside,
+                                           steps=args.steps, warmup=args.warmup)
     first = result["sizes"][args.sizes.split(",")[0]]
     line = {"metric": f"{design.capitalize()} beside {result['beside'].capitalize()} at equal size: prefill and decode tokens/s",
             "unit": "tokens/s",
@@ -92,9 +93,10 @@ def main() -> int:
     ap.add_argument("--layers", type=int, default=None, help="run fewer layers than the 28 of the config")
     ap.add_argument("--no-points", action="store_true", help="skip batch 1 and 64")
     ap.add_argument("--no-e2e", action="store_true")
-    ap.add_argument("--workload", choices=sorted(WORKLOADS) + ["koronex", "dotivik", "tudasun", "rizovik", "zetenex"],
+    ap.add_argument("--workload", choices=sorted(WORKLOADS) + DESIGNS,
                     help="run a serving workload, or the two-architecture comparison, instead of the decode bench")
     ap.add_argument("--sizes", default="2k,4k", help="with a design as the workload: which sizes to time")
+    ap.add_argument("--beside", choices=DESIGNS + ["qwen2"], help="with a design as the workload: set it beside this model")
     ap.add_argument("--graph-after", type=int, default=8,
                     help="with --workload: capture a decode graph at the N-th step that asks for it")
     args = ap.parse_args()
@@ -106,7 +108,7 @@ def main() -> int:
     if args.impl == "reference":
         return reference_arm(args)
     args.warmup = max(args.warmup, 3)
-    if args.workload in ("koronex", "dotivik", "tudasun", "rizovik", "zetenex"):
+    if args.workload in DESIGNS:
         if args.steps == 64:
             args.steps = 32
         return compare(args)

@@ -504,6 +504,27 @@ def zetenex_shape(width: int, heads: int, kv_heads: int, head_dim: int, ff: int,
     return shape
 
 
+def rudutar_shape(width: int, heads: int, kv_heads: int, head_dim: int, ff: int, layers: int, vocab: int,
+                  window: int = 1024) -> dict:
+    """A Rudutar config.json of a real model's sizes: groups of three layers (windowed attention over convolved heads,
+    windowed attention whose values are the keys, attention that reads the first one's keys), the feed-forwards dense
+    (``ff`` wide) and routed in turn: 16 experts in 4 groups of which 2 are kept, 2 a token, each ff / 4 wide, beside a
+    shared expert ff / 2 wide, so that a token's products are as many as in the dense one."""
+    att = dict(heads=heads, kv_heads=kv_heads, dim=head_dim, vdim=head_dim, conv=4, scale=head_dim ** -0.5,
+               mask=dict(size=window), q_temp=dict(coef=0.1, every=1024))
+    key = dict(heads=heads, kv_heads=kv_heads, dim=head_dim, vdim=head_dim, scale=head_dim ** -0.5, mask=dict(size=window),
+               rot=dict(dims=head_dim // 2, base=10000.0))
+    moe = dict(kind="moe", expert=dict(ff=ff // 4), shared=dict(ff=ff // 2),
+               router=dict(experts=16, top=2, scale=1.5, groups=dict(count=4, keep=2)))
+    kinds = [("attention", att), ("attention_2", key), ("attention", att)]
+    out = []
+    for i in range(layers):
+        kind, mixer = kinds[i % 3]
+        mixer = dict(mixer, kv_from=i - 2) if i % 3 == 2 else dict(mixer)
+        out.append(dict(type=kind, mixer=mixer, mlp=dict(moe) if i % 2 else dict(kind="dense", ff=ff)))
+    return dict(architecture="Rudutar", vocab=vocab, width=width, norm=dict(eps=1e-5), layers=out)
+
+
 def qwen2_shape(width: int, heads: int, kv_heads: int, head_dim: int, ff: int, layers: int, vocab: int) -> dict:
     return dict(architectures=["Qwen2ForCausalLM"], model_type="qwen2", vocab_size=vocab, hidden_size=width,
                 intermediate_size=ff, num_hidden_layers=layers, num_attention_heads=heads,
@@ -680,14 +701,17 @@ COMPARE_SIZES = {
 
 
 DESIGN_SHAPES = {"koronex": koronex_shape, "dotivik": dotivik_shape, "tudasun": tudasun_shape, "rizovik": rizovik_shape,
-                 "zetenex": zetenex_shape, "qwen2": qwen2_shape}
+                 "zetenex": zetenex_shape, "rudutar": rudutar_shape, "qwen2": qwen2_shape}
 # the existing model that a design is set beside: Tudasun beside Koronex, the other design with a recurrent mixer over
 # a float32 state, softmax attention with a sink, layers that read another layer's rows and a per-layer token input
 # Rizovik beside Tudasun: routed feed-forwards, a recurrent mixer over a float32 state, attention over a cache that keeps
 # every row
 # Zetenex beside Koronex: a recurrence over a float32 state, softmax attention with a gate, a plain feed-forward (up,
 # activation, down)
-BESIDE = {"koronex": "qwen2", "dotivik": "qwen2", "tudasun": "koronex", "rizovik": "tudasun", "zetenex": "koronex"}
+# Rudutar beside Koronex: windowed attention with a sink and a gate, layers that read another layer's keys, a plain
+# feed-forward (its routed feed-forwards are like Tudasun's)
+BESIDE = {"koronex": "qwen2", "dotivik": "qwen2", "tudasun": "koronex", "rizovik": "tudasun", "zetenex": "koronex",
+          "rudutar": "koronex"}
 
 
 def compare_architectures(sizes=("2k", "4k"), design: str = "koronex", beside: str | None = None, **kw) -> dict:
