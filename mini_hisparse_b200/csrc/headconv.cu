@@ -78,18 +78,17 @@ __device__ __forceinline__ float temperature(const Args& a, int pos) {
     return a.temp_coef != 0.f ? 1.f + a.temp_coef * log1pf((float)floor((double)(pos + 1) / a.temp_every)) : 1.f;
 }
 
-// where a token's row of this head goes: a row of q_out, or a page's row (null: the table names no page of the pool)
-template <typename CT>
-__device__ __forceinline__ CT* target(const Args& a, const Head& h, int t, int seg, int pos, int lane) {
-    if (h.kind == 0) return (CT*)a.q_out + ((size_t)t * a.nq + h.index) * a.dk;
+// where a token's row of this head goes: its first element in q_out or in the pool (-1: the table names no page of the pool)
+__device__ __forceinline__ long long target(const Args& a, const Head& h, int t, int seg, int pos) {
+    if (h.kind == 0) return ((long long)t * a.nq + h.index) * a.dk;
     const int page = a.block_table[(size_t)seg * a.width + pos / a.P], within = pos % a.P;
     if (page < 0 || page >= a.num_pages) {          // never write outside the pool
-        if (lane == 0 && a.status) atomicOr(a.status, 2);
-        return nullptr;
+        if (a.status) atomicOr(a.status, 2);
+        return -1;
     }
-    CT* base = (CT*)a.cache + (size_t)page * ((size_t)a.nkv * a.P * (a.dk + a.dv));
-    if (h.kind == 1) return base + ((size_t)h.index * a.P + within) * a.dk;
-    return base + (size_t)a.nkv * a.P * a.dk + ((size_t)h.index * a.P + within) * a.dv;
+    const long long base = (long long)page * ((long long)a.nkv * a.P * (a.dk + a.dv));
+    if (h.kind == 1) return base + ((long long)h.index * a.P + within) * a.dk;
+    return base + (long long)a.nkv * a.P * a.dk + ((long long)h.index * a.P + within) * a.dv;
 }
 
 // ---- heads up to 128 wide, multiples of four, up to four taps --------------------------------------------------
@@ -142,34 +141,61 @@ window_kernel(const Args a) {
 #pragma unroll
             for (int r = 0; r < TAPS - 1; ++r) store4(kept + (size_t)r * a.C + c, raw(t1 - (TAPS - 1) + r));
     }
+    // lane l looks up where token begin + l goes and its temperature; the others ask it
+    long long my_row = -1;
+    float my_temp = 1.f;
+    if (lane < TILE && begin + lane < end) {
+        const int pos = a.positions[begin + lane];
+        my_row = target(a, h, begin + lane, seg, pos);
+        if (h.kind == 0) my_temp = temperature(a, pos);
+    }
+    CT* out = (CT*)(h.kind == 0 ? a.q_out : a.cache);
     for (int t = begin; t < end; t += AHEAD) {
-        float4 u[AHEAD];
+        float4 u[AHEAD], y[AHEAD];
+        float ss[AHEAD];
 #pragma unroll
         for (int i = 0; i < AHEAD; ++i) u[i] = inside && t + i < end ? raw(t + i) : zero;
 #pragma unroll
         for (int i = 0; i < AHEAD; ++i) {
-            if (t + i >= end) break;
-            float4 y = zero;
+            y[i] = zero;
             if (inside) {
 #pragma unroll
-                for (int j = 0; j < TAPS - 1; ++j) {
-                    y.x = fmaf(w[j].x, win[j].x, y.x); y.y = fmaf(w[j].y, win[j].y, y.y);
-                    y.z = fmaf(w[j].z, win[j].z, y.z); y.w = fmaf(w[j].w, win[j].w, y.w);
+                for (int j = 0; j < TAPS; ++j) {              // the window runs on into this round's tokens
+                    const int at = i + j - (TAPS - 1);
+                    const float4 v = at >= 0 ? u[at >= 0 ? at : 0] : win[at >= 0 ? 0 : TAPS - 1 + at];
+                    y[i].x = fmaf(w[j].x, v.x, y[i].x); y[i].y = fmaf(w[j].y, v.y, y[i].y);
+                    y[i].z = fmaf(w[j].z, v.z, y[i].z); y[i].w = fmaf(w[j].w, v.w, y[i].w);
                 }
-                y.x = fmaf(w[TAPS - 1].x, u[i].x, y.x); y.y = fmaf(w[TAPS - 1].y, u[i].y, y.y);
-                y.z = fmaf(w[TAPS - 1].z, u[i].z, y.z); y.w = fmaf(w[TAPS - 1].w, u[i].w, y.w);
             }
-            const int pos = a.positions[t + i];
-            if (h.kind < 2) {
-                const float ss = warp_sum(y.x * y.x + y.y * y.y + y.z * y.z + y.w * y.w);
-                const float f = (h.kind == 0 ? temperature(a, pos) : 1.f) / sqrtf(ss / (float)h.d + a.eps);
-                y.x *= f * gain.x; y.y *= f * gain.y; y.z *= f * gain.z; y.w *= f * gain.w;
-            }
-            CT* dst = target<CT>(a, h, t + i, seg, pos, lane);
-            if (dst && inside) store4(dst + e, y);
+            ss[i] = y[i].x * y[i].x + y[i].y * y[i].y + y[i].z * y[i].z + y[i].w * y[i].w;
+        }
+        if (h.kind < 2) {
 #pragma unroll
-            for (int j = 0; j + 1 < TAPS - 1; ++j) win[j] = win[j + 1];
-            if constexpr (TAPS > 1) win[TAPS - 2] = u[i];
+            for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+                for (int i = 0; i < AHEAD; ++i) ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], o);
+        }
+#pragma unroll
+        for (int i = 0; i < AHEAD; ++i) {
+            const int from = (t + i - begin) & 31;
+            const long long row = __shfl_sync(0xffffffffu, my_row, from);
+            const float temp = __shfl_sync(0xffffffffu, my_temp, from);
+            if (h.kind < 2) {
+                const float f = temp / sqrtf(ss[i] / (float)h.d + a.eps);
+                y[i].x *= f * gain.x; y[i].y *= f * gain.y; y[i].z *= f * gain.z; y[i].w *= f * gain.w;
+            }
+            if (t + i < end && row >= 0 && inside) store4(out + row + e, y[i]);
+        }
+        if constexpr (TAPS > 1) {                             // the window after the last token of this round that exists
+            const int n = min(AHEAD, end - t);
+#pragma unroll
+            for (int i = 0; i < AHEAD; ++i) {
+#pragma unroll
+                for (int j = 0; j < TAPS - 1; ++j) {
+                    const float4 next = j + 1 < TAPS - 1 ? win[j + 1 < TAPS - 1 ? j + 1 : 0] : u[i];
+                    if (i < n) win[j] = next;
+                }
+            }
         }
     }
     if constexpr (TAPS > 1) {
@@ -226,8 +252,9 @@ general_kernel(const Args a) {
             f = (h.kind == 0 ? temperature(a, pos) : 1.f) / sqrtf(warp_sum(ss) / (float)h.d + a.eps);
             g = h.kind == 0 ? a.q_weight : a.k_weight;
         }
-        CT* dst = target<CT>(a, h, t, seg, pos, lane);
-        if (dst)
+        const long long at = target(a, h, t, seg, pos);
+        CT* dst = (CT*)(h.kind == 0 ? a.q_out : a.cache) + (at >= 0 ? at : 0);
+        if (at >= 0)
             for (int e = lane; e < h.d; e += 32) dst[e] = from_float<CT>(row[e] * (f * (g ? g[e] : 1.f)));
     }
     if (first && R > 0) {

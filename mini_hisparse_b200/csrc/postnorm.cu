@@ -23,6 +23,7 @@ namespace {
 
 __device__ __forceinline__ float load_parts(const float* p, size_t idx, int nsplit, size_t split_stride) {
     float v = p[idx];
+#pragma unroll 4
     for (int s = 1; s < nsplit; ++s) v += p[idx + (size_t)s * split_stride];
     return v;
 }
@@ -447,7 +448,7 @@ MHB_EXPORT int mhb_qknorm_rope_append_opts(const float* qkv, int nsplit, long lo
     MHB_DISPATCH_DTYPE(dtype, CT, {
         auto kern = qknorm_rope_append_kernel<CT, CT>;
         if (allow_smem(kern, smem, "qknorm_rope_append")) return -1;
-        launch_kernel(kern, dim3(T), dim3(row_threads(qw + kw)), smem, stream, qkv, nsplit, (size_t)split_stride, ld,
+        launch_kernel(kern, dim3(T), dim3(T <= 64 && qw + kw > 512 ? 1024 : row_threads(qw + kw)), smem, stream, qkv, nsplit, (size_t)split_stride, ld,
                       q_weight, k_weight, eps, positions, tok_seg, block_table, table_width, inv_freq, rdim,
                       (CT*)q_out, (CT*)cache, nq, nkv, dk, dv, P, num_pages, has_kv, status, per_head, v_eps,
                       (size_t)page_extra, temp_coef, temp_every, v_scale, bias, v_from_k);
