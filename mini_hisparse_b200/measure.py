@@ -539,7 +539,7 @@ class KernelTimes:
     SKIP = {"stream_scope", "dtype_code", "stream_k_scratch", "gemm_tc_wait_limit", "KernelError",
             "attention_decode_supports", "attention_tma_supports", "gemm_tc_qkv_rope_supports",
             "attention_decode_max_clusters", "lightning_chunk_smem", "c_double", "attention_mma_ext_supports",
-            "lightning_chunked_tc_supports"}
+            "lightning_chunked_tc_supports", "moe_plan_words", "moe_max_tiles"}
 
     def __enter__(self):
         self.saved, self.events = {}, []
